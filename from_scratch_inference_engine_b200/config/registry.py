@@ -13,6 +13,7 @@ import json
 from pathlib import Path
 from typing import Any, Dict, Mapping, Type
 
+from .deginex import DeginexConfig
 from .kufulix import KufulixConfig
 from .metulix import MetulixConfig
 from .qwen2 import ConfigError, Qwen2Config
@@ -84,3 +85,4 @@ register_architecture("Metulix", MetulixConfig)
 register_architecture("Zadepel", ZadepelConfig)
 register_architecture("Tapalix", TapalixConfig)
 register_architecture("Kufulix", KufulixConfig)
+register_architecture("Deginex", DeginexConfig)

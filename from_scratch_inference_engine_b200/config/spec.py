@@ -89,6 +89,9 @@ class ModelSpec:
     inlets: Tuple[Tuple[PartSpec, str], ...] = ()      # (part, tensor-name prefix) per inlet
     embedding_norm: Optional[PartSpec] = None          # a norm on the embedding rows: its result is
     embedding_norm_prefix: str = ""                    # the residual stream the first layer meets
+    streams: int = 0                       # > 0: the residual is this many streams, all equal to the
+                                           # embedding output at the start and summed at the end
+                                           # (arrangements that wire several streams, such as "streams")
 
     def resolved_schedule(self) -> List[Tuple[int, int, bool]]:
         """(layer, cache entry, writes) per call with defaults filled in and checked."""

@@ -57,6 +57,8 @@ LIBRARIES: Dict[str, Sequence[str]] = {
     # outputs, the residual stream beside the embedding output, capped logits, a sigmoid gate; and a
     # feed-forward of routed experts
     "routed": ("parallel_norm.cu", "routed.cu"),
+    # residuals of several streams that every sublayer reads and writes through small matrices
+    "streams": ("stream_norm.cu",),
 }
 # specialisations compiled by build_all() beside the default form of every library
 DEFAULT_SPECIALISATIONS = {"attn_mma": [("-DHEAD_DIM=128",)],

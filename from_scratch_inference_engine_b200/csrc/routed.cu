@@ -5,7 +5,9 @@
 //              experts form `groups` equal groups of neighbours, a group's score is the sum of its two
 //              largest choices, only experts of the `keep` best groups can be chosen (the others
 //              count as minus infinity); the `top` largest choices are taken; their weights are
-//              s / (sum of the chosen s + 1e-20) * scale (normalise = 0: s * scale)
+//              s / (sum of the chosen s + 1e-20) * scale (normalise = 0: s * scale).  With a router
+//              bias z = W_r y + bias.  Scores over the chosen alone: s = z for the choice, and the
+//              weights are softmax(z) over the chosen experts * scale
 //   align      (token, choice) pairs sorted by expert, cut into tiles of rows that share an expert
 //   gate_up    act[r] = f(W_gate[e] y[t(r)]) * (W_up[e] y[t(r)])       r in sorted order
 //   down       out[pair(r)] = W_down[e] act[r]
@@ -21,6 +23,9 @@
 namespace fsie {
 
 constexpr int MOE_TILE = 64;          // rows (and output columns) per tile of the tiled products
+
+// what a router's logits become: sigmoid, softmax over all experts, softmax over the chosen ones
+enum { SCORES_SIGMOID = 0, SCORES_SOFTMAX = 1, SCORES_CHOSEN_SOFTMAX = 2 };
 
 // -------------------------------------------------------------------------------- router
 // (value, index) maximum over a shared array by one warp; ties go to the lower index.
@@ -45,9 +50,10 @@ __device__ __forceinline__ int warp_argmax(const float* v, const unsigned char* 
 template <typename T>
 __global__ void moe_route_kernel(const T* __restrict__ y, int y_ld, const float* __restrict__ w_router,
                                  const float* __restrict__ logits,
-                                 const float* __restrict__ correction, int* __restrict__ ids,
-                                 float* __restrict__ weights, int width, int experts, int top, int groups,
-                                 int keep, float scale, int softmax_scores, int normalise, int group_max) {
+                                 const float* __restrict__ bias, const float* __restrict__ correction,
+                                 int* __restrict__ ids, float* __restrict__ weights, int width, int experts,
+                                 int top, int groups, int keep, float scale, int score_kind, int normalise,
+                                 int group_max) {
     extern __shared__ float route_smem[];
     float* row = route_smem;                       // [width]
     float* score = row + width;                    // [experts] s
@@ -67,14 +73,14 @@ __global__ void moe_route_kernel(const T* __restrict__ y, int y_ld, const float*
             float acc = 0.f;
             for (int c = lane; c < width; c += 32) acc = fmaf(wr[c], row[c], acc);
             acc = warp_sum(acc);
-            if (lane == 0) score[e] = acc;
+            if (lane == 0) score[e] = acc + (bias ? bias[e] : 0.f);
         }
     } else {
-        for (int e = threadIdx.x; e < experts; e += blockDim.x) score[e] = logits[(size_t)t * experts + e];
+        for (int e = threadIdx.x; e < experts; e += blockDim.x) score[e] = logits[(size_t)t * experts + e] + (bias ? bias[e] : 0.f);
     }
     __syncthreads();
     if (warp != 0) return;
-    if (softmax_scores) {
+    if (score_kind == SCORES_SOFTMAX) {
         float m = -INFINITY;
         for (int e = lane; e < experts; e += 32) m = fmaxf(m, score[e]);
         m = warp_max(m);
@@ -82,7 +88,7 @@ __global__ void moe_route_kernel(const T* __restrict__ y, int y_ld, const float*
         for (int e = lane; e < experts; e += 32) sum += expf(score[e] - m);
         sum = warp_sum(sum);
         for (int e = lane; e < experts; e += 32) score[e] = expf(score[e] - m) / sum;
-    } else {
+    } else if (score_kind == SCORES_SIGMOID) {
         for (int e = lane; e < experts; e += 32) score[e] = 1.0f / (1.0f + expf(-score[e]));
     }
     for (int e = lane; e < experts; e += 32) {
@@ -112,7 +118,7 @@ __global__ void moe_route_kernel(const T* __restrict__ y, int y_ld, const float*
             if (!group_taken[e / per]) taken[e] = 1;       // outside the kept groups: never chosen
         __syncwarp();
     }
-    float sum = 0.f;
+    float sum = 0.f, largest = -INFINITY;
     for (int k = 0; k < top; ++k) {
         const int e = warp_argmax(choice, taken, experts, lane);
         if (lane == 0) {
@@ -120,9 +126,16 @@ __global__ void moe_route_kernel(const T* __restrict__ y, int y_ld, const float*
             if (e >= 0) taken[e] = 1;
         }
         sum += e < 0 ? 0.f : score[e];
+        if (e >= 0) largest = fmaxf(largest, score[e]);
         __syncwarp();
     }
-    if (lane == 0) {
+    if (score_kind == SCORES_CHOSEN_SOFTMAX) {
+        if (lane != 0) return;
+        float total = 0.f;
+        for (int k = 0; k < top; ++k) total += expf(score[ids[(size_t)t * top + k]] - largest);
+        for (int k = 0; k < top; ++k)
+            weights[(size_t)t * top + k] = expf(score[ids[(size_t)t * top + k]] - largest) / total * scale;
+    } else if (lane == 0) {
         for (int k = 0; k < top; ++k) {
             const float s = score[ids[(size_t)t * top + k]];
             weights[(size_t)t * top + k] = normalise ? s / (sum + 1e-20f) * scale : s * scale;
@@ -483,15 +496,15 @@ extern "C" {
 
 int fsie_moe_tile_rows() { return MOE_TILE; }
 
-// y [tokens, y_ld] of the storage type; w_router float32 [experts, width]; correction float32
+// y [tokens, y_ld] of the storage type; w_router float32 [experts, width]; bias and correction float32
 // [experts] or null; ids int32 / weights float32 [tokens, top].
-int fsie_moe_route(const void* y, int y_ld, const float* w_router, const float* logits, const float* correction, int* ids,
-                   float* weights, int tokens, int width, int experts, int top, int groups, int keep,
-                   float scale, int softmax_scores, int normalise, int group_max, int dtype,
+int fsie_moe_route(const void* y, int y_ld, const float* w_router, const float* logits, const float* bias,
+                   const float* correction, int* ids, float* weights, int tokens, int width, int experts, int top,
+                   int groups, int keep, float scale, int score_kind, int normalise, int group_max, int dtype,
                    cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if ((y && width <= 0) || experts <= 0 || top <= 0 || top > experts || groups <= 0 || experts % groups ||
-        keep <= 0 || keep > groups || top > keep * (experts / groups))
+        score_kind < SCORES_SIGMOID || score_kind > SCORES_CHOSEN_SOFTMAX || keep <= 0 || keep > groups || top > keep * (experts / groups))
         return ERR_BAD_ARGUMENT;
     if (!y && !logits) return ERR_BAD_ARGUMENT;
     if (!y) width = 0;
@@ -502,13 +515,13 @@ int fsie_moe_route(const void* y, int y_ld, const float* w_router, const float* 
         if (smem > 48 * 1024)
             cudaFuncSetAttribute(moe_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         return launch_dependent(moe_route_kernel<float>, tokens, threads, smem, stream, (const float*)y, y_ld, w_router,
-                                logits, correction, ids, weights, width, experts, top, groups, keep, scale,
-                                softmax_scores, normalise, group_max);
+                                logits, bias, correction, ids, weights, width, experts, top, groups, keep, scale,
+                                score_kind, normalise, group_max);
     }
     if (smem > 48 * 1024)
         cudaFuncSetAttribute(moe_route_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     return launch_dependent(moe_route_kernel<bf16>, tokens, threads, smem, stream, (const bf16*)y, y_ld, w_router,
-                            logits, correction, ids, weights, width, experts, top, groups, keep, scale, softmax_scores,
+                            logits, bias, correction, ids, weights, width, experts, top, groups, keep, scale, score_kind,
                             normalise, group_max);
 }
 

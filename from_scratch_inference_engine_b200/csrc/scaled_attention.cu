@@ -6,7 +6,9 @@
 //
 //   s_h(i, j) = (q_h,i . k_g(h),j) * head_scale[h]      visible: j <= i and (window == 0 or i - j < window)
 //                                                       and (chunk == 0 or i / chunk == j / chunk)
+//   softcap > 0:  s_h(i, j) <- softcap * tanh(s_h(i, j) / softcap)
 //   o_h,i     = sum_j softmax_j(s_h(i, .)) v_g(h),j      g(h) = h / (heads / kv_heads)
+//   with gates:   o_h,i <- o_h,i * sigmoid(gate_h,i)     column by column, before the result is rounded
 //
 // Work is cut as in attention_generic.cu: a tile is up to ROWS query rows of one request and one
 // key/value head, a row being (token, head of the group): row = token * group + head_in_group; a
@@ -38,6 +40,8 @@ struct ScaledAttnParams {
     float* part_o; float* part_ml;            // [nsplit, tokens, heads, value_dim], [nsplit, tokens, heads, 2]
     int tokens, heads, kv_heads, window, nsplit;
     int chunk;                                // > 0: a query sees only the keys of its own chunk of this many positions
+    float softcap;                            // > 0: scores pass through softcap * tanh(s / softcap)
+    const void* gate; int gate_ld;            // null, or head h of token t at t * gate_ld + h * value_dim
     int* error;
 };
 
@@ -47,6 +51,14 @@ __device__ __forceinline__ int sa_first_key(const ScaledAttnParams& p, int pos) 
     if (p.chunk > 0) first = max(first, pos - pos % p.chunk);
     return max(first, 0);
 }
+
+// softcap * tanh(s / softcap) through one exponential: tanh(x) = 1 - 2 / (1 + e^(2x)), which ends at
+// +-1 where the exponential over- or underflows.  The error is a few 32-bit roundings of softcap.
+__device__ __forceinline__ float sa_cap_fast(float s, float cap, float twice_inv) {
+    return cap - __fdividef(2.0f * cap, 1.0f + __expf(s * twice_inv));
+}
+
+__device__ __forceinline__ float sa_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 template <typename T, int DPL, bool SHARED_V>
 __global__ void __launch_bounds__(SA_WARPS * 32) scaled_attention_kernel(const ScaledAttnParams p) {
@@ -157,6 +169,10 @@ __global__ void __launch_bounds__(SA_WARPS * 32) scaled_attention_kernel(const S
                 s[i] = fmaf(qq.w, k3v, s[i]);
             }
         }
+        if (p.softcap > 0.f) {
+#pragma unroll
+            for (int i = 0; i < SA_RPW; ++i) s[i] = p.softcap * tanhf(s[i] / p.softcap);
+        }
         float pj[SA_RPW];
         bool any = false;
 #pragma unroll
@@ -202,7 +218,10 @@ __global__ void __launch_bounds__(SA_WARPS * 32) scaled_attention_kernel(const S
 #pragma unroll
             for (int c = 0; c < DPL; ++c) {
                 const int d = lane + 32 * c;
-                if (d < dv) o[d] = from_float<T>(acc[i][c] * inv);
+                if (d >= dv) continue;
+                float v = acc[i][c] * inv;
+                if (p.gate) v *= sa_sigmoid(to_float(((const T*)p.gate)[(size_t)tok * p.gate_ld + (size_t)h * dv + d]));
+                o[d] = from_float<T>(v);
             }
         } else {
             const size_t idx = ((size_t)split * p.tokens + tok) * p.heads + h;
@@ -252,6 +271,16 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src, bool vali
 }
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+
+// two neighbouring columns of a result, times the sigmoid of their gates where there are any
+__device__ __forceinline__ __nv_bfloat162 sa_gated_pair(float a, float b, const bf16* gate) {
+    if (gate) {
+        const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gate));
+        a *= sa_sigmoid(z.x);
+        b *= sa_sigmoid(z.y);
+    }
+    return __floats2bfloat162_rn(a, b);
+}
 
 struct MmaLayout {
     int ldk, ldv, ldp;
@@ -364,6 +393,7 @@ __global__ void __launch_bounds__(SA_WARPS * 32) scaled_attention_mma_kernel(con
         sc[i] = r < nrows ? p.head_scale[kvh * group + (row0 + r) % group] : 0.f;
         m[i] = -INFINITY; l[i] = 0.f;
     }
+    const float cap_inv = p.softcap > 0.f ? 2.0f / p.softcap : 0.f;
     float acc[NV][4];
 #pragma unroll
     for (int n = 0; n < NV; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
@@ -404,7 +434,9 @@ __global__ void __launch_bounds__(SA_WARPS * 32) scaled_attention_mma_kernel(con
                 const int j = vi * 16 + n * 8 + 2 * t + (e & 1);
                 const int kj = k0 + j;
                 seen[n][e] = kj < kend && kj <= pos[i] && kj >= first_key[i];
-                s[n][e] = seen[n][e] ? s[n][e] * sc[i] : -INFINITY;
+                float sv = s[n][e] * sc[i];
+                if (p.softcap > 0.f) sv = sa_cap_fast(sv, p.softcap, cap_inv);
+                s[n][e] = seen[n][e] ? sv : -INFINITY;
                 tmax[i] = fmaxf(tmax[i], s[n][e]);
             }
 #pragma unroll
@@ -491,10 +523,11 @@ __global__ void __launch_bounds__(SA_WARPS * 32) scaled_attention_mma_kernel(con
         if (p.nsplit == 1) {
             const float inv = total > 0.f ? 1.0f / total : 0.f;
             bf16* o = (bf16*)p.out + (size_t)tok * p.out_ld + (size_t)h * dv + vi * dvq + 2 * t;
+            const bf16* gr = p.gate ? (const bf16*)p.gate + (size_t)tok * p.gate_ld + (size_t)h * dv + vi * dvq + 2 * t : nullptr;
 #pragma unroll
             for (int n = 0; n < NV; ++n)
                 *reinterpret_cast<__nv_bfloat162*>(o + n * 8) =
-                    __floats2bfloat162_rn(acc[n][2 * i] * inv, acc[n][2 * i + 1] * inv);
+                    sa_gated_pair(acc[n][2 * i] * inv, acc[n][2 * i + 1] * inv, gr ? gr + n * 8 : nullptr);
         } else {
             const size_t idx = ((size_t)split * p.tokens + tok) * p.heads + h;
             float* o = p.part_o + idx * dv + vi * dvq + 2 * t;
@@ -620,6 +653,7 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
     const int warp_rows = min(16, nrows - warp * 16);
     const int warp_last = warp_rows > 0 ? pos0 + (row0 + warp * 16 + warp_rows - 1) / group : -1;
     const int warp_first = warp_rows > 0 ? pos0 + (row0 + warp * 16) / group : 0;
+    const float cap_inv = p.softcap > 0.f ? 2.0f / p.softcap : 0.f;
     float acc[NVT][4];
 #pragma unroll
     for (int n = 0; n < NVT; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
@@ -658,12 +692,22 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
 #pragma unroll
         for (int n = 0; n < 8; ++n)
 #pragma unroll
+            for (int e = 0; e < 4; ++e) s[n][e] *= sc[e >> 1];
+        if (p.softcap > 0.f) {
+#pragma unroll
+            for (int n = 0; n < 8; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[n][e] = sa_cap_fast(s[n][e], p.softcap, cap_inv);
+        }
+#pragma unroll
+        for (int n = 0; n < 8; ++n)
+#pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int i = e >> 1;
                 const int j = n * 8 + 2 * t + (e & 1);
                 const int kj = k0 + j;
                 const bool seen = kj < kend && kj <= pos[i] && kj >= first_key[i];
-                s[n][e] = seen ? s[n][e] * sc[i] : -INFINITY;
+                if (!seen) s[n][e] = -INFINITY;
                 tmax[i] = fmaxf(tmax[i], s[n][e]);
             }
         float corr[2];
@@ -726,10 +770,11 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
         if (p.nsplit == 1) {
             const float inv = l[i] > 0.f ? 1.0f / l[i] : 0.f;
             bf16* o = (bf16*)p.out + (size_t)tok * p.out_ld + (size_t)h * dv + 2 * t;
+            const bf16* gr = p.gate ? (const bf16*)p.gate + (size_t)tok * p.gate_ld + (size_t)h * dv + 2 * t : nullptr;
 #pragma unroll
             for (int n = 0; n < NVT; ++n)
                 *reinterpret_cast<__nv_bfloat162*>(o + n * 8) =
-                    __floats2bfloat162_rn(acc[n][2 * i] * inv, acc[n][2 * i + 1] * inv);
+                    sa_gated_pair(acc[n][2 * i] * inv, acc[n][2 * i + 1] * inv, gr ? gr + n * 8 : nullptr);
         } else {
             const size_t idx = ((size_t)split * p.tokens + tok) * p.heads + h;
             float* o = p.part_o + idx * dv + 2 * t;
@@ -745,8 +790,10 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
 template <typename T>
 __global__ void sa_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                   T* __restrict__ out, int out_ld, int tokens, int heads, int dv,
-                                  int nsplit) {
+                                  int nsplit, const T* __restrict__ gate, int gate_ld) {
     const int tok = blockIdx.x, h = blockIdx.y;
+    grid_dependency_wait();
+    grid_dependents_go();
     float mmax = -INFINITY;
     for (int z = 0; z < nsplit; ++z)
         mmax = fmaxf(mmax, part_ml[(((size_t)z * tokens + tok) * heads + h) * 2]);
@@ -764,7 +811,9 @@ __global__ void sa_combine_kernel(const float* __restrict__ part_o, const float*
             const float mz = part_ml[idx * 2];
             if (mz != -INFINITY) o += part_o[idx * dv + d] * expf(mz - mmax);
         }
-        out[(size_t)tok * out_ld + (size_t)h * dv + d] = from_float<T>(o * inv);
+        o *= inv;
+        if (gate) o *= sa_sigmoid(to_float(gate[(size_t)tok * gate_ld + (size_t)h * dv + d]));
+        out[(size_t)tok * out_ld + (size_t)h * dv + d] = from_float<T>(o);
     }
 }
 
@@ -833,7 +882,8 @@ __global__ void rotate_mix_write_kernel(T* __restrict__ proj, int ld, const int*
 // One block per token of proj = [ q (heads x dim) | k (kv_heads x dim) | v (kv_heads x vdim) | ... ],
 // a warp per head of q and k in turn.
 //   q, k   with gains (q_gain, k_gain [dim], shared by the heads): every head divided by its root
-//          mean square (eps inside the root) times the gain, in 32-bit, BEFORE the rotation;
+//          mean square (eps inside the root) times the gain, in 32-bit, BEFORE the rotation; with
+//          `unit` a side without a gain is divided by its root mean square alone;
 //          then pairs (i, i + rotary_dim / 2) turn by the token's angles; q in place, k into its page
 //   v      into its page as it is
 template <typename T>
@@ -843,7 +893,7 @@ __global__ void norm_rotate_write_kernel(T* __restrict__ proj, int ld, const int
                                          T* __restrict__ v_pages, long long page_stride, int page_size,
                                          int heads, int kv_heads, int dim, int vdim, int rotary_dim,
                                          const float* __restrict__ q_gain, const float* __restrict__ k_gain,
-                                         float eps, int* __restrict__ error) {
+                                         float eps, int unit, int* __restrict__ error) {
     extern __shared__ float nr_smem[];                 // [warps][dim]
     const int t = blockIdx.x;
     grid_dependency_wait();
@@ -872,9 +922,9 @@ __global__ void norm_rotate_write_kernel(T* __restrict__ proj, int ld, const int
             mine[d] = v;
             sq += v * v;
         }
-        if (gain) {
+        if (gain || unit) {
             const float inv = 1.0f / sqrtf(warp_sum(sq) / (float)dim + eps);
-            for (int d = lane; d < dim; d += 32) mine[d] = mine[d] * inv * gain[d];
+            for (int d = lane; d < dim; d += 32) mine[d] = gain ? mine[d] * inv * gain[d] : mine[d] * inv;
         }
         __syncwarp();
         T* dst = is_q ? src : k_pages + page * page_stride + ((long long)(h - heads) * page_size + off) * dim;
@@ -987,6 +1037,7 @@ static bool scaled_attention_mma_takes(const ScaledAttnParams& p, int dtype, boo
         return false;
     if (p.page_stride % 8 || p.q_ld % 8 || p.out_ld % 2 || p.value_ld % 8) return false;
     if (((size_t)p.q | (size_t)p.k_pages | (size_t)p.v_pages) & 15 || ((size_t)p.out & 3)) return false;
+    if (p.gate && (p.gate_ld % 2 || ((size_t)p.gate & 3))) return false;
     return MmaLayout(p.key_dim, dv, shared_v).total <= 227 * 1024;
 }
 
@@ -1012,19 +1063,20 @@ int fsie_scaled_attention_tile_rows(int dtype, int key_dim, int value_dim, int v
 // 32-bit kernel; 2: a tensor-core kernel or refusal; 3: the tensor-core kernel whose warps split the
 // value columns, or refusal.  The tiles hold fsie_scaled_attention_tile_rows(...) rows.
 // With nsplit > 1 the caller gives part_o [nsplit, tokens, heads, value_dim] and part_ml
-// [nsplit, tokens, heads, 2] (float); the ranges are merged after the launch.
+// [nsplit, tokens, heads, 2] (float); the ranges are merged after the launch.  softcap 0: no cap on
+// the scores; gate null, or heads x value_dim columns per token of the storage type, rows gate_ld apart.
 int fsie_scaled_attention(const void* q, int q_ld, const float* head_scale, const void* k_pages,
                           const void* v_pages, long long page_stride, int page_size, int key_dim,
                           int value_dim, int values_in_keys, const int* block_tables, int bt_stride,
                           const int* tile_item, const int* tile_row0, int tiles, const int* item_qstart,
                           const int* item_qlen, const int* item_pos0, const int* item_slots, void* out,
                           int out_ld, float* part_o, float* part_ml, int tokens, int heads, int kv_heads,
-                          int window, int chunk, int nsplit, int dtype, int form, int* error,
-                          cudaStream_t stream) {
+                          int window, int chunk, float softcap, const void* gate, int gate_ld, int nsplit,
+                          int dtype, int form, int* error, cudaStream_t stream) {
     if (tokens <= 0 || tiles <= 0) return 0;
     if (tiles > 65535 || nsplit > 65535) return ERR_UNSUPPORTED;
     if (key_dim <= 0 || value_dim <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || nsplit < 1 ||
-        page_size <= 0 || window < 0 || chunk < 0 || (values_in_keys && value_dim > key_dim))
+        page_size <= 0 || window < 0 || chunk < 0 || !(softcap >= 0.f) || (values_in_keys && value_dim > key_dim))
         return ERR_BAD_ARGUMENT;
     if (nsplit > 1 && (!part_o || !part_ml)) return ERR_BAD_ARGUMENT;
     ScaledAttnParams p;
@@ -1037,7 +1089,7 @@ int fsie_scaled_attention(const void* q, int q_ld, const float* head_scale, cons
     p.item_qstart = item_qstart; p.item_qlen = item_qlen; p.item_pos0 = item_pos0; p.item_slots = item_slots;
     p.out = out; p.out_ld = out_ld; p.part_o = part_o; p.part_ml = part_ml;
     p.tokens = tokens; p.heads = heads; p.kv_heads = kv_heads; p.window = window; p.nsplit = nsplit;
-    p.chunk = chunk;
+    p.chunk = chunk; p.softcap = softcap; p.gate = gate; p.gate_ld = gate_ld;
     p.error = error;
     int rc;
     const int tile_rows = fsie_scaled_attention_tile_rows(dtype, key_dim, value_dim, values_in_keys, form);
@@ -1069,10 +1121,10 @@ int fsie_scaled_attention(const void* q, int q_ld, const float* head_scale, cons
     const dim3 cgrid(tokens, heads);
     const int threads = value_dim >= 128 ? 128 : (value_dim >= 64 ? 64 : 32);
     if (dtype == DTYPE_F32)
-        sa_combine_kernel<float><<<cgrid, threads, 0, stream>>>(part_o, part_ml, (float*)out, out_ld, tokens, heads, value_dim, nsplit);
-    else
-        sa_combine_kernel<bf16><<<cgrid, threads, 0, stream>>>(part_o, part_ml, (bf16*)out, out_ld, tokens, heads, value_dim, nsplit);
-    return FSIE_LAUNCH_CHECK();
+        return launch_dependent(sa_combine_kernel<float>, cgrid, dim3(threads), 0, stream, part_o, part_ml, (float*)out,
+                                out_ld, tokens, heads, value_dim, nsplit, (const float*)gate, gate_ld);
+    return launch_dependent(sa_combine_kernel<bf16>, cgrid, dim3(threads), 0, stream, part_o, part_ml, (bf16*)out,
+                            out_ld, tokens, heads, value_dim, nsplit, (const bf16*)gate, gate_ld);
 }
 
 // proj [tokens, ld] = q | k | v head by head; cos_sin [table_len, rotary_dim]; slot_of [tokens]
@@ -1100,13 +1152,13 @@ int fsie_rotate_mix_write(void* proj, int ld, const int* positions, const float*
 
 
 // proj [tokens, ld] = q | k | v head by head (more columns may follow); q_gain / k_gain [dim] float or
-// null (no norm of that side); cos_sin [table_len, rotary_dim]; slot_of [tokens] (page * page_size +
+// null (no norm of that side, or - unit != 0 - a norm without a gain); cos_sin [table_len, rotary_dim]; slot_of [tokens] (page * page_size +
 // offset, -1: store nothing).
 int fsie_norm_rotate_write(void* proj, int ld, const int* positions, const float* cos_sin, int table_len,
                            const int* slot_of, void* k_pages, void* v_pages, long long page_stride,
                            int page_size, int tokens, int heads, int kv_heads, int dim, int vdim,
-                           int rotary_dim, const float* q_gain, const float* k_gain, float eps, int dtype,
-                           int* error, cudaStream_t stream) {
+                           int rotary_dim, const float* q_gain, const float* k_gain, float eps, int unit,
+                           int dtype, int* error, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (rotary_dim < 0 || rotary_dim > dim || (rotary_dim & 1) || dim <= 0 ||
         ld < (heads + kv_heads) * dim + kv_heads * vdim)
@@ -1118,11 +1170,11 @@ int fsie_norm_rotate_write(void* proj, int ld, const int* positions, const float
         return launch_dependent(norm_rotate_write_kernel<float>, dim3(tokens), dim3(warps * 32), smem, stream,
                                 (float*)proj, ld, positions, cos_sin, table_len, slot_of, (float*)k_pages,
                                 (float*)v_pages, page_stride, page_size, heads, kv_heads, dim, vdim, rotary_dim,
-                                q_gain, k_gain, eps, error);
+                                q_gain, k_gain, eps, unit, error);
     return launch_dependent(norm_rotate_write_kernel<bf16>, dim3(tokens), dim3(warps * 32), smem, stream,
                             (bf16*)proj, ld, positions, cos_sin, table_len, slot_of, (bf16*)k_pages,
                             (bf16*)v_pages, page_stride, page_size, heads, kv_heads, dim, vdim, rotary_dim,
-                            q_gain, k_gain, eps, error);
+                            q_gain, k_gain, eps, unit, error);
 }
 
 // out [tokens, out_ld] holds heads x vdim columns per token, gate [tokens, gate_ld] one column per head.

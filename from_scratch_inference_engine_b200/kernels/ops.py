@@ -1300,9 +1300,9 @@ def mixers():
         lib.fsie_scaled_attention_tile_rows.argtypes = [i, i, i, i, i]
         lib.fsie_scaled_attention_tile_rows.restype = i
         lib.fsie_scaled_attention.argtypes = [p, i, p, p, p, ll, i, i, i, i, p, i, p, p, i, p, p, p, p,
-                                              p, i, p, p, i, i, i, i, i, i, i, i, p, p]
+                                              p, i, p, p, i, i, i, i, i, f, p, i, i, i, i, p, p]
         lib.fsie_norm_rotate_write.argtypes = [p, i, p, p, i, p, p, p, ll, i, i, i, i, i, i, i, p, p, f,
-                                               i, p, p]
+                                               i, i, p, p]
         lib.fsie_head_gate.argtypes = [p, i, p, i, i, i, i, i, p]
         lib.fsie_scaled_sum_rmsnorm.argtypes = [p, p, f, p, f, p, p, p, i, i, f, i, i, p]
         lib.fsie_rotate_mix_write.argtypes = [p, i, p, p, i, p, p, p, ll, i, i, i, i, i, i, i, i, p, p,
@@ -1414,12 +1414,15 @@ def scaled_attention(q: torch.Tensor, q_ld: int, head_scale: torch.Tensor, k_pag
                      kv_heads: int, window: int, error: torch.Tensor, nsplit: int = 1,
                      part_o: Optional[torch.Tensor] = None,
                      part_ml: Optional[torch.Tensor] = None, form: str = "auto",
-                     chunk: int = 0) -> torch.Tensor:
+                     chunk: int = 0, softcap: float = 0.0,
+                     gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal (optionally windowed; `chunk` > 0: only over the keys j with j // chunk == i // chunk)
     softmax attention of q [tokens, heads x key_dim] over paged keys
     [kv_head][slot][key_dim] and values [kv_head][slot][value_dim] (or, values_in_keys, the first
-    value_dim columns of the key rows), scores multiplied by head_scale[head]; scores, softmax and
-    weights in 32-bit.  `form`: "auto" takes a tensor-core kernel where one fits (bfloat16, key
+    value_dim columns of the key rows), scores multiplied by head_scale[head] and - `softcap` > 0 -
+    passed through softcap * tanh(. / softcap); scores, softmax and weights in 32-bit.  `gate`
+    [tokens, heads x value_dim] (may be a view of columns of a wider tensor): the result is multiplied
+    by its sigmoid column by column before it is rounded.  `form`: "auto" takes a tensor-core kernel where one fits (bfloat16, key
     sizes in steps of 16, value sizes 64 ... 512), "plain" the 32-bit kernel, "mma" insists on a
     tensor-core kernel, "mma_split" on the one whose warps split the value columns.  The tiles
     hold `scaled_attention_rows(dtype, key_dim, value_dim, values_in_keys, form)` rows."""
@@ -1430,6 +1433,12 @@ def scaled_attention(q: torch.Tensor, q_ld: int, head_scale: torch.Tensor, k_pag
         raise KernelError("scaled_attention: cache dtype differs from q")
     if head_scale.numel() != heads or out.numel() < tokens * heads * value_dim:
         raise KernelError("scaled_attention: shapes do not fit")
+    gate_ld = 0
+    if gate is not None:
+        _need(gate, q.dtype, "gate", contiguous=False)
+        if gate.shape != (tokens, heads * value_dim) or gate.stride(1) != 1:
+            raise KernelError("scaled_attention: gate is not of the result's shape")
+        gate_ld = gate.stride(0)
     if nsplit > 1:
         if part_o.numel() < nsplit * tokens * heads * value_dim or \
                 part_ml.numel() < nsplit * tokens * heads * 2:
@@ -1439,7 +1448,7 @@ def scaled_attention(q: torch.Tensor, q_ld: int, head_scale: torch.Tensor, k_pag
         value_dim, int(values_in_keys), _ptr(block_tables), block_tables.stride(0), _ptr(tile_item),
         _ptr(tile_row0), tiles, _ptr(item_qstart), _ptr(item_qlen), _ptr(item_pos0), _ptr(item_slots),
         _ptr(out), heads * value_dim, _ptr(part_o), _ptr(part_ml), tokens, heads, kv_heads, window,
-        int(chunk), nsplit, _tag(q.dtype), SCALED_ATTENTION_FORMS[form], _ptr(error), _stream()),
+        int(chunk), float(softcap), _ptr(gate), gate_ld, nsplit, _tag(q.dtype), SCALED_ATTENTION_FORMS[form], _ptr(error), _stream()),
         "scaled_attention")
     return out
 
@@ -1478,9 +1487,10 @@ def norm_rotate_write(proj: torch.Tensor, positions: torch.Tensor, cos_sin: torc
                       slot_of: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
                       page_stride: int, page_size: int, heads: int, kv_heads: int, dim: int, vdim: int,
                       rotary_dim: int, q_gain: Optional[torch.Tensor], k_gain: Optional[torch.Tensor],
-                      eps: float, error: torch.Tensor) -> None:
+                      eps: float, error: torch.Tensor, unit: bool = False) -> None:
     """proj [tokens, q | k | v | ...]: every head of q (of k) divided by its root mean square (eps
-    inside the root) times q_gain (k_gain) [dim] in 32-bit where that gain is given; then q rotated in
+    inside the root) times q_gain (k_gain) [dim] in 32-bit where that gain is given (`unit`: where it is
+    not given, divided by its root mean square alone); then q rotated in
     place and k into its page over the first rotary_dim of each head (pairs i, i + rotary_dim / 2);
     values into their page."""
     _need(proj, None, "proj")
@@ -1500,8 +1510,8 @@ def norm_rotate_write(proj: torch.Tensor, positions: torch.Tensor, cos_sin: torc
     _check(mixers().fsie_norm_rotate_write(_ptr(proj), ld, _ptr(positions), _ptr(cos_sin), cos_sin.shape[0],
                                            _ptr(slot_of), _ptr(k_pages), _ptr(v_pages), page_stride,
                                            page_size, tokens, heads, kv_heads, dim, vdim, rotary_dim,
-                                           _ptr(q_gain), _ptr(k_gain), float(eps), _tag(proj.dtype),
-                                           _ptr(error), _stream()), "norm_rotate_write")
+                                           _ptr(q_gain), _ptr(k_gain), float(eps), int(unit),
+                                           _tag(proj.dtype), _ptr(error), _stream()), "norm_rotate_write")
 
 
 def head_gate(out: torch.Tensor, gate: torch.Tensor, heads: int, vdim: int) -> torch.Tensor:
@@ -1607,7 +1617,7 @@ def routed():
         lib.fsie_logit_cap.argtypes = [p, ll, f, f, p]
         lib.fsie_sigmoid_gate.argtypes = [p, i, p, i, i, i, i, p]
         lib.fsie_moe_tile_rows.argtypes = []
-        lib.fsie_moe_route.argtypes = [p, i, p, p, p, p, p, i, i, i, i, i, i, f, i, i, i, i, p]
+        lib.fsie_moe_route.argtypes = [p, i, p, p, p, p, p, p, i, i, i, i, i, i, f, i, i, i, i, p]
         lib.fsie_moe_align.argtypes = [p, i, i, i, i, p, p, p, p, p, p, p]
         lib.fsie_moe_gather.argtypes = [p, ll, p, p, i, i, p, i, i, p]
         lib.fsie_moe_product.argtypes = [p, ll, p, p, ll, p, p, p, p, p, i, i, i, i, i, i, i, i, p]
@@ -1703,6 +1713,9 @@ def sigmoid_gate(out: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
     return out
 
 
+ROUTER_SCORES = {"sigmoid": 0, "softmax": 1, "chosen_softmax": 2}
+
+
 def moe_tile_rows() -> int:
     return routed().fsie_moe_tile_rows()
 
@@ -1710,18 +1723,21 @@ def moe_tile_rows() -> int:
 def moe_route(y: Optional[torch.Tensor], w_router: Optional[torch.Tensor], correction: Optional[torch.Tensor],
               ids: torch.Tensor, weights: torch.Tensor, top: int, groups: int, keep: int, scale: float,
               scores: str = "sigmoid", normalise: bool = True, logits: Optional[torch.Tensor] = None,
-              group_score: str = "top2") -> None:
+              group_score: str = "top2", bias: Optional[torch.Tensor] = None) -> None:
     """Per token: s = sigmoid (or softmax) of the router's logits in 32-bit; the `top` experts with the
     largest s + correction among the `keep` best of `groups` groups (a group's score: the sum of its
     two largest s + correction, or - `group_score` "max" - the largest); weights s / (their sum + 1e-20) * scale.  The logits are w_router y, summed here
     (w_router float32 [experts, width]) or - `logits`, float32 [tokens, experts] - by a product
-    before this call.  ids int32, weights float32, both [tokens, top]."""
+    before this call; `bias` (float32 [experts]) is added to them.  `scores` "chosen_softmax": the choice
+    is made on the logits (+ correction), the weights are the logits' softmax over the chosen experts
+    alone, times scale.  ids int32, weights float32, both [tokens, top]."""
     _need(ids, torch.int32, "ids")
     _need(weights, torch.float32, "weights")
-    if correction is not None:
-        _need(correction, torch.float32, "correction")
-    if scores not in ("sigmoid", "softmax"):
-        raise KernelError("moe_route: scores must be 'sigmoid' or 'softmax'")
+    for name, vector in (("correction", correction), ("bias", bias)):
+        if vector is not None:
+            _need(vector, torch.float32, name)
+    if scores not in ROUTER_SCORES:
+        raise KernelError(f"moe_route: scores must be one of {', '.join(ROUTER_SCORES)}")
     if group_score not in ("top2", "max"):
         raise KernelError("moe_route: group_score must be 'top2' or 'max'")
     if logits is not None:
@@ -1737,11 +1753,11 @@ def moe_route(y: Optional[torch.Tensor], w_router: Optional[torch.Tensor], corre
             raise KernelError("moe_route: shapes do not fit")
         y_ptr, y_ld, tag, w_ptr = _ptr(y), y.stride(0), _tag(y.dtype), _ptr(w_router)
     if ids.numel() < tokens * top or weights.numel() < tokens * top or \
-            (correction is not None and correction.numel() != experts):
+            any(vector is not None and vector.numel() != experts for vector in (correction, bias)):
         raise KernelError("moe_route: shapes do not fit")
-    _check(routed().fsie_moe_route(y_ptr, y_ld, w_ptr, _ptr(logits), _ptr(correction), _ptr(ids),
-                                   _ptr(weights), tokens, width, experts, int(top), int(groups), int(keep),
-                                   float(scale), int(scores == "softmax"), int(normalise),
+    _check(routed().fsie_moe_route(y_ptr, y_ld, w_ptr, _ptr(logits), _ptr(bias), _ptr(correction),
+                                   _ptr(ids), _ptr(weights), tokens, width, experts, int(top), int(groups),
+                                   int(keep), float(scale), ROUTER_SCORES[scores], int(normalise),
                                    int(group_score == "max"), tag, _stream()), "moe_route")
 
 
@@ -1845,4 +1861,69 @@ def moe_combine(expert_out: torch.Tensor, weights: torch.Tensor, shared: Optiona
     _check(routed().fsie_moe_combine(_ptr(expert_out), _ptr(weights), _ptr(shared), _ptr(place), _ptr(out),
                                      tokens, width, int(top), _ptr(ids), int(experts), _ptr(y), y_ld,
                                      _tag(out.dtype), _stream()), "moe_combine")
+    return out
+
+
+# ------------------------------------------------------------------ a residual of several streams
+_streams = None
+
+
+def streams_lib():
+    """The library of residuals of several streams, compiled at first use."""
+    global _streams
+    if _streams is None:
+        lib = build.load_library("streams")
+        i, f, p = ctypes.c_int, ctypes.c_float, ctypes.c_void_p
+        lib.fsie_stream_norm.argtypes = [p, p, p, p, p, p, p, p, p, p, i, i, i, f, i, i, i, p]
+        lib.fsie_stream_norm.restype = i
+        _streams = lib
+    return _streams
+
+
+def stream_norm(x: torch.Tensor, start: Optional[torch.Tensor], delta: Optional[torch.Tensor],
+                mix: Optional[torch.Tensor], spread: Optional[torch.Tensor], gather: Optional[torch.Tensor],
+                gain: Optional[torch.Tensor], bias: Optional[torch.Tensor], eps: float,
+                out: Optional[torch.Tensor], rows: Optional[torch.Tensor] = None, write_x: bool = True,
+                centred: bool = True) -> Optional[torch.Tensor]:
+    """x (float32 [tokens, streams, width]) holds a token's streams; with `start` (float32 [tokens,
+    width]) they do not exist yet and every one equals the token's row of it.  A pending sublayer
+    output `delta` [tokens, width] settles first: x_t <- sum_r mix[r, t] x_r + spread[t] delta for all
+    streams at once (mix [streams, streams], spread [streams], float32).  Then out = norm of
+    sum_t gather[t] x_t (gather None: the plain sum), `centred` a layer norm (gain, bias), else an RMS
+    norm, in out's dtype.  Without `out` only the settling.  With `rows` (int32 indices) only those
+    rows, into out[0..len(rows)); x is left untouched unless write_x."""
+    _need(x, torch.float32, "x")
+    tokens, streams, width = x.shape
+    dtype = out.dtype if out is not None else (delta.dtype if delta is not None else None)
+    if dtype is None:
+        raise KernelError("stream_norm: nothing to do")
+    if start is not None:
+        _need(start, torch.float32, "start")
+        if start.shape != (tokens, width):
+            raise KernelError("stream_norm: start is not one row per token")
+    if delta is not None:
+        _need(delta, dtype, "delta")
+        _need(mix, torch.float32, "mix")
+        _need(spread, torch.float32, "spread")
+        if delta.shape != (tokens, width) or mix.shape != (streams, streams) or spread.numel() != streams:
+            raise KernelError("stream_norm: the pending output or its coefficients do not fit")
+    if gather is not None:
+        _need(gather, torch.float32, "gather")
+        if gather.numel() != streams:
+            raise KernelError("stream_norm: one gather coefficient per stream")
+    count = tokens
+    if rows is not None:
+        _need(rows, torch.int32, "rows")
+        count = rows.numel()
+    if out is not None:
+        _need(out, None, "out")
+        _need(gain, torch.float32, "gain")
+        if bias is not None:
+            _need(bias, torch.float32, "bias")
+        if gain.numel() != width or (bias is not None and bias.numel() != width) or out.numel() < count * width:
+            raise KernelError("stream_norm: gain, bias or out does not fit")
+    _check(streams_lib().fsie_stream_norm(_ptr(x), _ptr(start), _ptr(delta), _ptr(mix), _ptr(spread), _ptr(gather),
+                                          _ptr(gain), _ptr(bias), _ptr(rows), _ptr(out), count, streams, width,
+                                          float(eps), int(write_x), int(centred), _tag(dtype), _stream()),
+           "stream_norm")
     return out

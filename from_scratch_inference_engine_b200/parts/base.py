@@ -14,7 +14,8 @@ and the cache come from the context.
     class FeedForward:    forward(ctx, y) -> [tokens, hidden]
     class Arrangement:    forward(ctx, x, delta, cache) -> delta'
                           (x is the float32 residual stream, updated in place; delta is
-                          the output of the previous sublayer not yet added to x)
+                          the output of the previous sublayer not yet added to x; in a model
+                          with several residual streams x is [tokens, streams, hidden])
     class Inlet:          forward(ctx, x, delta, x0) -> x'
                           (runs between two calls of the run order; x0 is the embedding output of
                           the step's tokens; nothing is left pending behind it)

@@ -10,7 +10,7 @@ from ..config.spec import LayerSpec
 from ..kernels import ops
 from ..weights.tensor_spec import TensorSpec
 from .base import LayerCache, Part, build_part, register_part
-from .norm import LayerNorm, NormedDelta, PendingSum, RMSNorm
+from .norm import LayerNorm, NormedDelta, PendingSum, RMSNorm, StreamNorm, StreamUpdate
 
 
 @register_part("arrangement", "prenorm")
@@ -254,3 +254,102 @@ class ParallelBlock(Part):
         if self.feed_forward is None:
             return PendingSum((mixed,))
         return PendingSum((mixed, self.feed_forward.forward(ctx, y)))
+
+
+class _StreamCoefficients:
+    """How one sublayer meets a residual of several streams: its input is sum_t gather[t] x_t, and its
+    output y changes every stream, x_t <- sum_r mix[r, t] x_r + spread[t] y."""
+
+    def __init__(self, prefix: str, streams: int, names):
+        self.streams = streams
+        self.names = {which: prefix + name for which, name in names.items()}
+        self.gather = self.mix = self.spread = None
+
+    def tensor_specs(self, optional: bool = False) -> List[TensorSpec]:
+        s = self.streams
+        return [TensorSpec(self.names["gather"], (s,), role="vector", init="gain", optional=optional),
+                TensorSpec(self.names["spread"], (s,), role="vector", init="gain", optional=optional),
+                TensorSpec(self.names["mix"], (s, s), role="vector", init="eye", optional=optional)]
+
+    def bind(self, tensors) -> None:
+        for which, name in self.names.items():
+            setattr(self, which, tensors[name].to(torch.float32).contiguous())
+
+
+@register_part("arrangement", "streams")
+class StreamsBlock(Part):
+    """A pre-norm layer on a residual of several streams x_1 .. x_s (hyper-connections), for each of
+    its two sublayers f: y = f(norm(sum_t gather[t] x_t)), then x_t <- sum_r mix[r, t] x_r + spread[t] y
+    for all streams at once from the old ones.  A layer may have no feed-forward.
+
+    The residual is float32 [tokens, streams, width].  A sublayer's output is not spread at once: it is
+    handed on with its coefficients (`StreamUpdate`), and the kernel of the norm that runs next - the
+    next sublayer's, or the model's final norm on the wanted rows only - spreads it, gathers the
+    streams and norms the gathered row in one pass.  The coefficients of sublayer q (1: mixer, 2:
+    feed-forward) are the tensors "hc<q>.in", "hc<q>.out" and "hc<q>.mix" below the layer's prefix;
+    `STREAM_NAMES` names them.
+    """
+
+    STREAM_NAMES = ({"gather": "hc1.in", "spread": "hc1.out", "mix": "hc1.mix"},
+                    {"gather": "hc2.in", "spread": "hc2.out", "mix": "hc2.mix"})
+
+    def __init__(self, prefix: str, layer: LayerSpec, streams: int):
+        if streams < 1:
+            raise ValueError("the streams arrangement needs a model with at least one stream")
+        self.prefix, self.streams = prefix, int(streams)
+        self.mixer_norm = build_part("norm", layer.mixer_norm, prefix + layer.mixer_norm_name)
+        self.mixer = build_part("mixer", layer.mixer, prefix + layer.mixer_name)
+        self.feed_forward = self.feed_forward_norm = None
+        self.coefficients = [_StreamCoefficients(prefix, self.streams, self.STREAM_NAMES[0])]
+        second = _StreamCoefficients(prefix, self.streams, self.STREAM_NAMES[1])
+        # a checkpoint may still hold the norm and the coefficients of a feed-forward that the layer
+        # does not have
+        self.unused: List[TensorSpec] = []
+        if layer.feed_forward is not None:
+            self.feed_forward_norm = build_part("norm", layer.feed_forward_norm,
+                                                prefix + layer.feed_forward_norm_name)
+            self.feed_forward = build_part("feed_forward", layer.feed_forward,
+                                           prefix + layer.feed_forward_name)
+            self.coefficients.append(second)
+        else:
+            import dataclasses
+            self.unused = second.tensor_specs(optional=True)
+            if layer.feed_forward_norm is not None:
+                norm = build_part("norm", layer.feed_forward_norm, prefix + layer.feed_forward_norm_name)
+                self.unused += [dataclasses.replace(spec, optional=True) for spec in norm.tensor_specs()]
+        for norm in (self.mixer_norm, self.feed_forward_norm):
+            if norm is not None and not isinstance(norm, StreamNorm):
+                raise TypeError("the streams arrangement takes norms that read several streams "
+                                "(layernorm, rmsnorm)")
+
+    def parts(self):
+        return [part for part in (self.mixer_norm, self.mixer, self.feed_forward_norm,
+                                  self.feed_forward) if part is not None]
+
+    @property
+    def capturable(self) -> bool:
+        return all(part.capturable for part in self.parts())
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        return [spec for part in self.parts() for spec in part.tensor_specs()] + \
+            [spec for c in self.coefficients for spec in c.tensor_specs()] + self.unused
+
+    def bind(self, tensors, runtime) -> None:
+        self.runtime = runtime
+        for part in self.parts():
+            part.bind(tensors, runtime)
+        for c in self.coefficients:
+            c.bind(tensors)
+
+    def forward(self, ctx, x: torch.Tensor, delta: StreamUpdate, cache: LayerCache) -> StreamUpdate:
+        ctx.residual_copy = None
+        first = self.coefficients[0]
+        y = self.mixer_norm.over_streams(x, delta, first.gather, tag="streams.mixer_in")
+        # until an output has settled, the streams are the rows they all start from
+        start = delta.start if delta.delta is None else None
+        delta = StreamUpdate(self.mixer.forward(ctx, y, cache), first.mix, first.spread, start)
+        if self.feed_forward is None:
+            return delta
+        second = self.coefficients[1]
+        y = self.feed_forward_norm.over_streams(x, delta, second.gather, tag="streams.feed_forward_in")
+        return StreamUpdate(self.feed_forward.forward(ctx, y), second.mix, second.spread)

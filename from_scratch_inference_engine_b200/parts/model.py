@@ -13,13 +13,15 @@ from ..kernels import ops
 from ..weights.loader import check_tensors, to_runtime_dtype
 from ..weights.tensor_spec import TensorSpec
 from .base import LayerCache, StateNeed, build_part
+from .norm import StreamNorm, StreamUpdate
 
 
 class DecoderModel:
     """Embedding (times `embedding_scale`, then through `embedding_norm` where the model has one)
     -> blocks in the order of `spec.schedule`, an inlet
     before the calls that name one -> final norm -> head, times `logit_scale`, capped by
-    `logit_softcap * tanh(. / logit_softcap)` where a cap is given.
+    `logit_softcap * tanh(. / logit_softcap)` where a cap is given.  With `spec.streams` the residual
+    is that many streams, every one the embedding output at the start; the final norm reads their sum.
 
     The run order is data: entry i of the schedule runs block `layer` on cache entry
     `cache` (its own by default).  A block named twice runs twice with the same weights;
@@ -31,12 +33,15 @@ class DecoderModel:
         self.spec = spec
         self.schedule = spec.resolved_schedule()
         self.blocks = [build_part("arrangement",
-                                  _arrangement_spec(layer), layer.prefix) for layer in spec.layers]
+                                  _arrangement_spec(layer, spec.streams), layer.prefix) for layer in spec.layers]
         self.final_norm = build_part("norm", spec.final_norm, spec.final_norm_prefix)
         self.embedding_norm = None if spec.embedding_norm is None else \
             build_part("norm", spec.embedding_norm, spec.embedding_norm_prefix)
         self.inlets = [build_part("inlet", part, prefix) for part, prefix in spec.inlets]
         self.inlet_before = [call.inlet for call in spec.schedule]
+        if spec.streams and (self.inlets or not isinstance(self.final_norm, StreamNorm)):
+            raise ValueError("a model of several residual streams takes no inlets, and a final norm that reads "
+                             "several streams")
         self.embedding: Optional[torch.Tensor] = None
         self.head: Optional[torch.Tensor] = None
         self.runtime = None
@@ -132,11 +137,15 @@ class DecoderModel:
             rows = rt.buffer("model.embedding_rows", ctx.num_tokens, hidden, torch.float32)
             ops.embed_gather(ctx.token_ids, self.embedding, rows, ctx.error, scale)
             x = self.embedding_norm.forward(rows, None, tag="model.residual", out_dtype=torch.float32)
+        delta = None
+        if self.spec.streams:             # every stream starts as x; they exist once a layer has changed them
+            delta = StreamUpdate(start=x)
+            x = rt.buffer("model.streams", ctx.num_tokens, self.spec.streams * hidden, torch.float32)
+            x = x.view(ctx.num_tokens, self.spec.streams, hidden)
         x0 = None
         if self.inlets:                   # the embedding output, for the inlets that read it
             x0 = rt.buffer("model.embedding_output", ctx.num_tokens, hidden, torch.float32)
             ops.embed_gather(ctx.token_ids, self.embedding, x0, ctx.error, scale)
-        delta = None
         ctx.residual_copy = None          # x in the compute dtype, where an arrangement keeps one
         for index, (layer, _, _) in enumerate(self.schedule):
             if self.inlet_before[index] is not None:
@@ -145,7 +154,10 @@ class DecoderModel:
             delta = self.blocks[layer].forward(ctx, x, delta, caches[index])
         if want_rows is None or want_rows.numel() == 0:
             return None
-        y = self.final_norm.forward(x, delta, rows=want_rows, write_x=False)
+        if self.spec.streams:
+            y = self.final_norm.over_streams(x, delta, None, rows=want_rows, write_x=False)
+        else:
+            y = self.final_norm.forward(x, delta, rows=want_rows, write_x=False)
         # the logits live where the last step's lived: whoever gets them reads them (or queues
         # what reads them on this stream) before the next step runs
         logits = rt.linear_f32_out(y, self.head, "model.logits")
@@ -154,9 +166,9 @@ class DecoderModel:
         return logits
 
 
-def _arrangement_spec(layer):
+def _arrangement_spec(layer, streams: int):
     from ..config.spec import PartSpec
-    return PartSpec(layer.arrangement, {"layer": layer})
+    return PartSpec(layer.arrangement, {"layer": layer, "streams": streams} if streams else {"layer": layer})
 
 
 def tensor_specs(spec: ModelSpec) -> List[TensorSpec]:

@@ -42,8 +42,39 @@ class ScaledSum:
     scales: tuple
 
 
+@dataclass
+class StreamUpdate:
+    """What is still to happen to a residual of several streams before the next sublayer reads it.
+    `start` (float32 [tokens, width]): the streams do not exist yet, every one equals these rows.
+    `delta`: a sublayer's output that is to be spread over the streams, x_t <- sum_r mix[r, t] x_r +
+    spread[t] delta (None: no sublayer has run)."""
+
+    delta: Optional[torch.Tensor] = None
+    mix: Optional[torch.Tensor] = None          # float32 [streams, streams], from x to
+    spread: Optional[torch.Tensor] = None       # float32 [streams]
+    start: Optional[torch.Tensor] = None
+
+
+class StreamNorm:
+    """Norms that can read a residual of several streams (a base of the norm parts below)."""
+
+    centred = False
+
+    def over_streams(self, x: torch.Tensor, pending: StreamUpdate, gather: Optional[torch.Tensor],
+                     rows: Optional[torch.Tensor] = None, write_x: bool = True,
+                     tag: Optional[str] = None) -> torch.Tensor:
+        """The normed rows of sum_t gather[t] x_t (gather None: the plain sum) in the compute dtype,
+        x float32 [tokens, streams, width]; what is pending settles first, in 32-bit and in the same
+        pass over the streams, and - with `write_x` - stays settled."""
+        gain, bias = self.stream_gain_bias()
+        count = x.shape[0] if rows is None else rows.numel()
+        out = self.runtime.buffer(tag, count, self.width, self.runtime.dtype)
+        return ops.stream_norm(x, pending.start, pending.delta, pending.mix, pending.spread, gather, gain, bias,
+                               self.eps, out, rows=rows, write_x=write_x, centred=self.centred)
+
+
 @register_part("norm", "rmsnorm")
-class RMSNorm(Part):
+class RMSNorm(StreamNorm, Part):
     """y = x * rsqrt(mean(x^2) + eps) * gain over the last axis, statistics in 32-bit (reference:
     src/model/nn.cpp:45-72, 64-bit statistics there).  The gain is the stored tensor, or - with
     `one_plus`, a weight stored around zero - 1 + the stored tensor (summed in 32-bit at bind).
@@ -79,6 +110,9 @@ class RMSNorm(Part):
             self._gain_f32 = self.gain.to(torch.float32).contiguous()
         return self._gain_f32
 
+    def stream_gain_bias(self):
+        return self.gain_f32, None
+
     def forward(self, x: torch.Tensor, delta: Union[None, torch.Tensor, NormedDelta, ScaledSum],
                 rows: Optional[torch.Tensor] = None, write_x: bool = True,
                 tag: Optional[str] = None, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
@@ -105,7 +139,7 @@ class RMSNorm(Part):
 
 
 @register_part("norm", "layernorm")
-class LayerNorm(Part):
+class LayerNorm(StreamNorm, Part):
     """y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * gain (+ bias) over the last axis,
     statistics in 32-bit.  The gain is `prefix + weight_name`; with `bias_name` there is a bias,
     the tensor `prefix + bias_name`.
@@ -117,6 +151,7 @@ class LayerNorm(Part):
     """
 
     capturable = True
+    centred = True
 
     def __init__(self, prefix: str, width: int, eps: float, weight_name: str = "weight",
                  bias_name: Optional[str] = None):
@@ -137,6 +172,9 @@ class LayerNorm(Part):
         self.gain = tensors[self.name].to(torch.float32).contiguous()
         if self.bias_name is not None:
             self.bias = tensors[self.bias_name].to(torch.float32).contiguous()
+
+    def stream_gain_bias(self):
+        return self.gain, self.bias
 
     def forward(self, x: torch.Tensor, delta: Union[None, torch.Tensor, PendingSum] = None,
                 rows: Optional[torch.Tensor] = None, write_x: bool = False,

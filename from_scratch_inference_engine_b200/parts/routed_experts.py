@@ -20,7 +20,9 @@ class RoutedExperts(Part):
     the experts', each an expert whose output is its input y itself (times its weight); they have
     no tensors, and they count as experts for the scores, the groups and the choice.
 
-    Router: z = W_r y in 32-bit, s = sigmoid(z) (`scores` "softmax": softmax over the experts).
+    Router: z = W_r y in 32-bit (`router_bias`: plus a stored vector), s = sigmoid(z) (`scores`
+    "softmax": softmax over the experts; "chosen_softmax": the choice is made on z itself, and the
+    weights are the softmax of z over the chosen experts alone, times `scale`).
     The choice is made on s + correction (a stored vector, `correction`=False: none) and the
     weights on s without it.  The experts form `groups` equal groups of neighbours; a group's
     score is the sum of its two largest choice values (`group_score` "max": the largest), and only
@@ -42,13 +44,14 @@ class RoutedExperts(Part):
     GROUPED_MIN_ROWS = 32       # average rows per expert from which the tcgen05 form is taken
 
     NAMES = {"expert": "e{index}.", "gate": "gate", "up": "up", "down": "down", "router": "router",
-             "correction": "correction", "shared": "shared."}
+             "correction": "correction", "shared": "shared.", "router_bias": "router.b"}
 
     def __init__(self, prefix: str, hidden_size: int, intermediate_size: int, experts: int, top: int,
                  groups: int = 1, keep: int = 1, scale: float = 1.0, scores: str = "sigmoid",
                  normalise: bool = True, correction: bool = True, activation: str = "silu",
                  shared: Optional[PartSpec] = None, names: Optional[Dict[str, str]] = None,
-                 gated: bool = True, identity: int = 0, group_score: str = "top2"):
+                 gated: bool = True, identity: int = 0, group_score: str = "top2",
+                 router_bias: bool = False):
         if activation not in (ops.FUSED_GATES if gated else ops.GATE_KINDS):
             raise ValueError(f"unknown activation '{activation}' for experts "
                              f"{'with' if gated else 'without'} a gate")
@@ -57,8 +60,8 @@ class RoutedExperts(Part):
         self.gated, self.identity, self.group_score = bool(gated), int(identity), group_score
         if self.identity < 0:
             raise ValueError("routed_experts: identity must not be negative")
-        if scores not in ("sigmoid", "softmax"):
-            raise ValueError("scores must be 'sigmoid' or 'softmax'")
+        if scores not in ops.ROUTER_SCORES:
+            raise ValueError(f"scores must be one of {', '.join(ops.ROUTER_SCORES)}")
         self.prefix, self.hidden_size = prefix, int(hidden_size)
         self.intermediate_size, self.experts, self.top = int(intermediate_size), int(experts), int(top)
         self.groups, self.keep, self.scale = int(groups), int(keep), float(scale)
@@ -71,12 +74,12 @@ class RoutedExperts(Part):
                              "keep in 1..groups")
         if self.top > self.keep * (self.routed // self.groups):
             raise ValueError("routed_experts: the kept groups hold fewer than `top` experts")
-        self.has_correction = bool(correction)
+        self.has_correction, self.has_router_bias = bool(correction), bool(router_bias)
         self.names = dict(self.NAMES)
         self.names.update(names or {})
         self.shared = None if shared is None else build_part("feed_forward", shared,
                                                              prefix + self.names["shared"])
-        self.w_router = self.correction = self.w_gate_up = self.w_down = None
+        self.w_router = self.router_bias = self.correction = self.w_gate_up = self.w_down = None
 
     @property
     def capturable(self) -> bool:
@@ -93,6 +96,8 @@ class RoutedExperts(Part):
                 specs.append(TensorSpec(self._expert(e, "gate"), (f, h)))
             specs += [TensorSpec(self._expert(e, "up"), (f, h)), TensorSpec(self._expert(e, "down"), (h, f))]
         specs.append(TensorSpec(self.prefix + self.names["router"], (self.routed, h)))     # in the compute dtype
+        if self.has_router_bias:
+            specs.append(TensorSpec(self.prefix + self.names["router_bias"], (self.routed,), role="vector"))
         if self.has_correction:
             specs.append(TensorSpec(self.prefix + self.names["correction"], (self.routed,), role="vector"))
         if self.shared is not None:
@@ -112,6 +117,8 @@ class RoutedExperts(Part):
                                    for e in range(self.experts)]).contiguous()
         self.w_router = tensors[self.prefix + self.names["router"]].contiguous()
         self._grouped = None             # descriptors of the stacked matrices, made when first needed
+        if self.has_router_bias:
+            self.router_bias = tensors[self.prefix + self.names["router_bias"]].to(torch.float32).contiguous()
         if self.has_correction:
             self.correction = tensors[self.prefix + self.names["correction"]].to(torch.float32).contiguous()
         if self.shared is not None:
@@ -132,7 +139,8 @@ class RoutedExperts(Part):
         weights = rt.buffer("routed.weights", tokens, top, torch.float32)
         logits = rt.linear_f32_out(y, self.w_router, "routed.logits")
         ops.moe_route(None, None, self.correction, ids, weights, top, self.groups, self.keep,
-                      self.scale, self.scores, self.normalise, logits=logits, group_score=self.group_score)
+                      self.scale, self.scores, self.normalise, logits=logits, group_score=self.group_score,
+                      bias=self.router_bias)
         # choices at or beyond `experts` are identity experts: no rows in the products, and the
         # weighted sum takes the token's own row for them
         identity = dict(ids=ids, experts=self.experts, y=y) if self.identity else {}

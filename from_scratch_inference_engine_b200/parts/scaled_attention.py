@@ -30,7 +30,8 @@ def key_splits(blocks: int, longest: int, sms: int, key_tile: int = 32) -> int:
 
 def attend(ctx, rt, q: torch.Tensor, head_scale: torch.Tensor, group, cache: LayerCache,
            out: torch.Tensor, heads: int, kv_heads: int, key_dim: int, value_dim: int,
-           values_in_keys: bool, window: int, chunk: int = 0) -> torch.Tensor:
+           values_in_keys: bool, window: int, chunk: int = 0, softcap: float = 0.0,
+           gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The step's tokens over the pages through `ops.scaled_attention`: tiles of query rows, key
     ranges split over blocks when the tiles are few."""
     tokens = q.shape[0]
@@ -38,7 +39,8 @@ def attend(ctx, rt, q: torch.Tensor, head_scale: torch.Tensor, group, cache: Lay
     value_ld = key_dim if values_in_keys else value_dim
     if form == "auto" and (q.stride(0) % 8 or cache.page_stride % 8 or value_ld % 8 or q.data_ptr() % 16
                            or cache.k_pages.data_ptr() % 16 or cache.v_pages.data_ptr() % 16
-                           or (heads * value_dim) % 2):
+                           or (heads * value_dim) % 2
+                           or (gate is not None and (gate.stride(0) % 2 or gate.data_ptr() % 4))):
         form = "plain"          # rows that do not start where the tensor-core kernels' 16-byte copies need them
     rows = ops.scaled_attention_rows(q.dtype, key_dim, value_dim, values_in_keys, form)
     tiles = ctx.attention_tiles(heads // kv_heads, rows)
@@ -55,15 +57,16 @@ def attend(ctx, rt, q: torch.Tensor, head_scale: torch.Tensor, group, cache: Lay
                                 values_in_keys, group.block_tables, tiles.item, tiles.row0,
                                 tiles.count, ctx.item_qstart, ctx.item_qlen, ctx.item_pos0,
                                 ctx.item_slots, out, tokens, heads, kv_heads, window, ctx.error,
-                                nsplit, part_o, part_ml, form=form, chunk=chunk)
+                                nsplit, part_o, part_ml, form=form, chunk=chunk, softcap=softcap,
+                                gate=gate)
 
 
 @register_part("mixer", "scaled_gqa_attention")
 class ScaledGqaAttention(Mixer):
-    """q, k, v projections with biases (one product over the stacked weight); rotation of q and
-    k by `position` (pairs i, i + rotary_dim / 2 over the first rotary_dim of a head); scores
+    """q, k, v projections with biases (`bias`=False: without; one product over the stacked weight);
+    rotation of q and k by `position` (pairs i, i + rotary_dim / 2 over the first rotary_dim of a head); scores
     (q . k) * scale * temperature[head] over the keys j <= i (or the last `window` of them);
-    softmax; head h reads key/value head h // (heads / kv_heads); output projection without bias.
+    with `softcap` > 0 then softcap * tanh(. / softcap); softmax; head h reads key/value head h // (heads / kv_heads); output projection without bias.
     Keys are `dim` wide, values `vdim`.
 
     `value_mix`: "source" keeps this layer's values of the step's tokens for later layers;
@@ -74,9 +77,11 @@ class ScaledGqaAttention(Mixer):
     `chunk` > 0: position i sees j <= i only where i // chunk == j // chunk, the chunks counted
     from position 0 of the sequence (beside, or instead of, the window).  `qk_norm`: every head of q
     and of k is divided by its root mean square (`eps` inside the root) times a stored gain of `dim`
-    numbers that all heads share, in 32-bit, before the rotation.  `head_gate`: every head's output
-    is multiplied by sigmoid(W_g y)[head], one number per head, before the output projection; W_g
-    rides in the one product with q, k and v.
+    numbers that all heads share, in 32-bit, before the rotation (`qk_gain`=False: no gain is stored,
+    the root mean square alone).  `head_gate`: every head's output is multiplied by
+    sigmoid(W_g y)[head], one number per head, before the output projection; `column_gate`: the
+    concatenated heads are multiplied element by element by sigmoid(W_g y), as the attention kernel
+    writes them.  W_g rides in the one product with q, k and v.
     `names` gives the tensor names below the prefix.
     """
 
@@ -89,7 +94,8 @@ class ScaledGqaAttention(Mixer):
                  vdim: int, scale: float, position: PartSpec, window: int = 0,
                  value_mix: str = "none", temperature: bool = True,
                  names: Optional[Dict[str, str]] = None, chunk: int = 0, qk_norm: bool = False,
-                 eps: float = 0.0, head_gate: bool = False):
+                 eps: float = 0.0, head_gate: bool = False, bias: bool = True, softcap: float = 0.0,
+                 qk_gain: bool = True, column_gate: bool = False):
         if heads % kv_heads:
             raise ValueError("heads must be a multiple of kv_heads")
         if value_mix not in ("none", "source", "mix"):
@@ -99,12 +105,17 @@ class ScaledGqaAttention(Mixer):
         self.scale, self.window, self.value_mix = float(scale), int(window), value_mix
         self.temperature = bool(temperature)
         self.chunk, self.qk_norm, self.eps, self.head_gate = int(chunk), bool(qk_norm), float(eps), bool(head_gate)
-        if self.chunk < 0 or self.window < 0:
-            raise ValueError("window and chunk must not be negative")
-        if (self.qk_norm or self.head_gate) and value_mix != "none":
-            raise ValueError("scaled_gqa_attention: blended values go with neither qk_norm nor head_gate")
+        self.bias, self.softcap, self.qk_gain = bool(bias), float(softcap), bool(qk_gain)
+        self.column_gate = bool(column_gate)
+        if self.chunk < 0 or self.window < 0 or self.softcap < 0:
+            raise ValueError("window, chunk and softcap must not be negative")
+        if self.head_gate and self.column_gate:
+            raise ValueError("scaled_gqa_attention: a gate per head or a gate per column, not both")
+        if (self.qk_norm or self.head_gate or self.column_gate) and value_mix != "none":
+            raise ValueError("scaled_gqa_attention: blended values go with neither qk_norm nor a gate")
         self.q_width, self.k_width = self.heads * self.dim, self.kv_heads * self.dim
         self.v_width = self.kv_heads * self.vdim
+        self.gate_width = self.heads if self.head_gate else (self.heads * self.vdim if self.column_gate else 0)
         self.position = build_part("position", position, prefix)
         if self.position.rotary_dim > self.dim:
             raise ValueError("the rotated size exceeds dim")
@@ -120,16 +131,17 @@ class ScaledGqaAttention(Mixer):
         specs = []
         for which, width in (("q", self.q_width), ("k", self.k_width), ("v", self.v_width)):
             specs.append(TensorSpec(p + n[which], (width, h)))
-            specs.append(TensorSpec(p + n[which] + n["bias"], (width,)))
+            if self.bias:
+                specs.append(TensorSpec(p + n[which] + n["bias"], (width,)))
         if self.value_mix != "none":        # the source has the tensor too, and does not use it
             specs.append(TensorSpec(p + n["mix"], (), role="vector", init="half"))
         if self.temperature:
             specs.append(TensorSpec(p + n["temperature"], (self.heads,), role="vector", init="gain"))
-        if self.qk_norm:
+        if self.qk_norm and self.qk_gain:
             specs += [TensorSpec(p + n[which] + n["norm"], (self.dim,), role="vector", init="gain")
                       for which in ("q", "k")]
-        if self.head_gate:
-            specs.append(TensorSpec(p + n["gate"], (self.heads, h)))
+        if self.gate_width:
+            specs.append(TensorSpec(p + n["gate"], (self.gate_width, h)))
         specs.append(TensorSpec(p + n["o"], (h, self.heads * self.vdim)))
         return specs + self.position.tensor_specs()
 
@@ -145,18 +157,20 @@ class ScaledGqaAttention(Mixer):
         self.runtime = runtime
         p, n = self.prefix, self.names
         stacked = [tensors[p + n[k]] for k in "qkv"]
-        biases = [tensors[p + n[k] + n["bias"]].to(runtime.dtype) for k in "qkv"]
-        if self.head_gate:                  # the gate's rows behind q, k and v; it has no bias
+        if self.gate_width:                 # the gate's rows behind q, k and v; it has no bias
             stacked.append(tensors[p + n["gate"]])
-            biases.append(torch.zeros(self.heads, dtype=runtime.dtype, device=biases[0].device))
         rows = sum(w.shape[0] for w in stacked)
-        if self.head_gate and rows % 8:     # rows of the product's result start on 16 bytes
+        if self.gate_width and rows % 8:    # rows of the product's result start on 16 bytes
             pad = 8 - rows % 8
             stacked.append(torch.zeros(pad, self.hidden_size, dtype=stacked[0].dtype, device=stacked[0].device))
-            biases.append(torch.zeros(pad, dtype=runtime.dtype, device=biases[0].device))
         self.w_qkv = torch.cat(stacked).contiguous()
-        self.b_qkv = torch.cat(biases).contiguous()
-        if self.qk_norm:
+        if self.bias:
+            biases = [tensors[p + n[k] + n["bias"]].to(runtime.dtype) for k in "qkv"]
+            behind = self.w_qkv.shape[0] - sum(b.numel() for b in biases)
+            if behind:
+                biases.append(torch.zeros(behind, dtype=runtime.dtype, device=biases[0].device))
+            self.b_qkv = torch.cat(biases).contiguous()
+        if self.qk_norm and self.qk_gain:
             self.q_gain = tensors[p + n["q"] + n["norm"]].to(torch.float32).contiguous()
             self.k_gain = tensors[p + n["k"] + n["norm"]].to(torch.float32).contiguous()
         self.w_o = tensors[p + n["o"]].contiguous()
@@ -186,20 +200,21 @@ class ScaledGqaAttention(Mixer):
             if v_first is None or v_first.shape != (tokens, self.v_width):
                 raise ValueError("scaled_gqa_attention: no layer before this one has left values "
                                  "of this width to blend with")
-        if self.qk_norm or self.head_gate:
+        if self.qk_norm or self.gate_width:
             ops.norm_rotate_write(qkv, ctx.positions, self.position.table, group.slot_of, cache.k_pages,
                                   cache.v_pages, cache.page_stride, group.page_size, self.heads,
                                   self.kv_heads, self.dim, self.vdim, self.position.rotary_dim,
-                                  self.q_gain, self.k_gain, self.eps, ctx.error)
+                                  self.q_gain, self.k_gain, self.eps, ctx.error, unit=self.qk_norm)
         else:
             ops.rotate_mix_write(qkv, ctx.positions, self.position.table, group.slot_of, cache.k_pages,
                                  cache.v_pages, cache.page_stride, group.page_size, self.heads,
                                  self.kv_heads, self.dim, self.vdim, self.position.rotary_dim, mode,
                                  self.mix, v_first, ctx.error)
         out = rt.buffer("scaled_attention.out", tokens, self.heads * self.vdim, qkv.dtype)
+        gate0 = self.q_width + self.k_width + self.v_width
+        gate = qkv[:, gate0:gate0 + self.gate_width] if self.gate_width else None
         attend(ctx, rt, qkv, self.head_scale, group, cache, out, self.heads, self.kv_heads, self.dim,
-               self.vdim, False, self.window, self.chunk)
+               self.vdim, False, self.window, self.chunk, self.softcap, gate if self.column_gate else None)
         if self.head_gate:
-            gate0 = self.q_width + self.k_width + self.v_width
-            ops.head_gate(out, qkv[:, gate0:gate0 + self.heads], self.heads, self.vdim)
+            ops.head_gate(out, gate, self.heads, self.vdim)
         return rt.linear(out, self.w_o, None, "scaled_attention.o")

@@ -26,7 +26,10 @@ feed-forward, depth and window (prefill of one prompt, decode steps of a batch, 
 `--workload zadepel` does the same for the Zadepel design (latent attention, grouped-query attention with
 blended values, minGRU) beside Qwen2 with full causal attention; `--workload kufulix` measures the
 Kufulix design (windowed attention beside a state-space mixer, chunked attention with gated heads, experts
-without gates) beside a Metulix model of equal size; `--workload tapalix` measures the
+without gates) beside a Metulix model of equal size; `--workload deginex` measures the Deginex design (a
+residual of four streams, chunked attention with unit q and k, capped scores and a gate per column, dense
+and routed feed-forwards in turn, a looped stretch) beside a Kufulix model of chunked attention layers of
+equal size; `--workload tapalix` measures the
 Tapalix design (latent attention with and without a rotated part, routed experts beside a shared one,
 a looped stretch of layers) beside a Zadepel model of latent attention layers with a dense feed-forward
 of the width a token uses, at equal depth.
@@ -521,6 +524,41 @@ def kufulix_shapes(width, heads, kv_heads, dim, ss_heads, ss_vdim, state, expert
     return kufulix, metulix
 
 
+# Deginex beside a Kufulix model: (name, width, heads, kv heads, head dim, streams, dense ff, experts, top,
+# expert ff, layers, passes over the middle layers, vocab)
+DEGINEX_SIZES = (("w2048", 2048, 16, 4, 128, 4, 6144, 32, 4, 1024, 4, 2, 32000),
+                 ("w4096", 4096, 32, 8, 128, 4, 12288, 16, 2, 2048, 4, 2, 32000))
+
+
+def deginex_shapes(width, heads, kv_heads, dim, streams, dense, experts, top, ff, layers, times, vocab, chunk):
+    """A Deginex model (dense and routed feed-forwards in turn, the middle layers run `times` times) and
+    the closest model the engine had: a Kufulix model of chunked attention layers in the same run order
+    (a later pass runs the first one's tensors), its experts - which have no gate - half as wide again so
+    that their matrices hold as many numbers, a dense layer as a single expert of that kind."""
+    attention = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                 "mask": {"size": chunk}}
+    mixer = dict(attention, softcap=30.0)
+    mlps = ({"kind": "dense", "ff": dense},
+            {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}})
+    loop = (1, layers - 1, times)
+    deginex = {"architecture": "Deginex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+               "streams": streams, "loop": dict(zip(("start", "stop", "times"), loop)),
+               "layers": [{"type": "attention", "mixer": mixer, "mlp": mlps[i % 2]} for i in range(layers)]}
+    plain = [{"kind": "moe", "expert": {"ff": dense * 3 // 2}, "router": {"experts": 1, "top": 1}},
+             {"kind": "moe", "expert": {"ff": ff * 3 // 2}, "router": {"experts": experts, "top": top}}]
+    order = list(range(loop[0])) + list(range(*loop[:2])) * times + list(range(loop[1], layers))
+    runs, first = [], {}
+    for run, i in enumerate(order):
+        layer = {"type": "attention", "mlp": plain[i % 2],
+                 "mixer": dict(attention, rot={"base": 10000.0, "dims": dim})}
+        if i in first:
+            layer["weights_of"] = first[i]
+        first.setdefault(i, run)
+        runs.append(layer)
+    kufulix = {"architecture": "Kufulix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": runs}
+    return deginex, kufulix
+
+
 def hybrid_workload(args, design="metulix") -> int:
     """The Metulix design (or, `design`, the Zadepel design) beside the Qwen2 model of equal size
     (random bf16 weights): prefill of
@@ -559,7 +597,7 @@ def hybrid_workload(args, design="metulix") -> int:
                                "sum_layernorm", "settle_concat", "logit_cap", "sigmoid_gate", "moe_route",
                                "moe_align", "moe_gather", "moe_product", "gemm_tiles_grouped", "moe_combine",
                                "ssd_prep", "ssd_tails", "ssd_gate_norm", "norm_rotate_write", "head_gate",
-                               "scaled_sum_rmsnorm")
+                               "scaled_sum_rmsnorm", "stream_norm")
              if hasattr(ops, name)]
 
     def by_kind(fn):
@@ -595,7 +633,7 @@ def hybrid_workload(args, design="metulix") -> int:
         out["(whole step)"] = total
         return {k: round(v, 4) for k, v in sorted(out.items(), key=lambda kv: -kv[1])}
 
-    table = {"tapalix": TAPALIX_SIZES, "kufulix": KUFULIX_SIZES}.get(design, HYBRID_SIZES)
+    table = {"tapalix": TAPALIX_SIZES, "kufulix": KUFULIX_SIZES, "deginex": DEGINEX_SIZES}.get(design, HYBRID_SIZES)
     sizes = [s for s in table if not args.sizes or s[0] in args.sizes.split(",")]
     results = []
     clocks = ClockSampler()
@@ -622,6 +660,16 @@ def hybrid_workload(args, design="metulix") -> int:
                      "experts": experts, "identity": identity, "top": top, "groups": [groups, keep],
                      "expert_ff": ff, "layers": layers, "vocab": vocab, "window": window, "chunk": 2 * window}
             beside = "metulix"
+        elif design == "deginex":
+            (name, width, heads, kv_heads, dim, streams, dense, experts, top, ff, layers, times, vocab) = size
+            layers = args.layers or layers
+            shapes = deginex_shapes(width, heads, kv_heads, dim, streams, dense, experts, top, ff, layers,
+                                    times, vocab, 2 * window)
+            entry = {"size": name, "width": width, "heads": heads, "kv_heads": kv_heads, "head_dim": dim,
+                     "streams": streams, "dense_ff": dense, "experts": experts, "top": top, "expert_ff": ff,
+                     "layers": layers, "passes": times, "layer_runs": len(shapes[1]["layers"]), "vocab": vocab,
+                     "chunk": 2 * window}
+            beside = "kufulix"
         else:
             name, width, heads, kv_heads, dim, ff, layers, vocab = size
             layers = args.layers or layers
@@ -697,7 +745,7 @@ def hybrid_workload(args, design="metulix") -> int:
     clock_record = clocks.stop()
     print(json.dumps({
         "metric": f"prefill and decode tokens/s of the {design.capitalize()} design beside "
-                  f"{ {'tapalix': 'Zadepel', 'kufulix': 'Metulix'}.get(design, 'Qwen2') } at equal size",
+                  f"{ {'tapalix': 'Zadepel', 'kufulix': 'Metulix', 'deginex': 'Kufulix'}.get(design, 'Qwen2') } at equal size",
         "impl": "engine", "unit": "tokens/s", "n_gpus": 1, "steps": steps, "warmup": warmup,
         "dtype": "bf16" if compute == "bfloat16" else "fp32",
         "config": {"prefill_tokens": prompt_len, "decode_batch": batch, "decode_context": context,
@@ -787,13 +835,16 @@ def main() -> int:
                              "blocks it falls to instead of sharing it out among all (for measuring that choice)")
     parser.add_argument("--fp32-steps", type=int, default=8,
                         help="decode steps timed on the float32 path after the bf16 run (0 = skip)")
-    parser.add_argument("--workload", default="decode", choices=["decode", "serving", "long", "timeline", "hybrid", "zadepel", "tapalix", "kufulix"],
+    parser.add_argument("--workload", default="decode", choices=["decode", "serving", "long", "timeline", "hybrid", "zadepel", "tapalix", "kufulix",
+                                                                        "deginex"],
                         help="decode: the default measurement; serving: continuous batching of 256 "
                              "requests at the 1.5B shape; long: the 14B shape, decode at batch 32 with "
                              "8,192-token contexts and chunked prefill of an 8,192-token prompt; "
                              "timeline: kernel start and end times inside one decode step (text); "
                              "hybrid: the Metulix design beside Qwen2 at equal sizes, prefill and decode; "
                              "zadepel: the same for the Zadepel design; "
+                             "kufulix: the Kufulix design beside a Metulix model; "
+                             "deginex: the Deginex design beside a Kufulix model of chunked attention layers; "
                              "tapalix: the Tapalix design beside a Zadepel model of latent attention layers")
     parser.add_argument("--sizes", default="", help="hybrid: which sizes to run (w2048,w4096; '' = all)")
     parser.add_argument("--requests", type=int, default=256)
@@ -824,6 +875,8 @@ def main() -> int:
         return hybrid_workload(args, design="tapalix")
     if args.workload == "kufulix":
         return hybrid_workload(args, design="kufulix")
+    if args.workload == "deginex":
+        return hybrid_workload(args, design="deginex")
 
     import numpy as np
     import torch

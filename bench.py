@@ -597,7 +597,7 @@ def hybrid_workload(args, design="metulix") -> int:
                                "sum_layernorm", "settle_concat", "logit_cap", "sigmoid_gate", "moe_route",
                                "moe_align", "moe_gather", "moe_product", "gemm_tiles_grouped", "moe_combine",
                                "ssd_prep", "ssd_tails", "ssd_gate_norm", "norm_rotate_write", "head_gate",
-                               "scaled_sum_rmsnorm", "stream_norm")
+                               "scaled_sum_rmsnorm", "stream_norm", "attention_tc_scaled")
              if hasattr(ops, name)]
 
     def by_kind(fn):

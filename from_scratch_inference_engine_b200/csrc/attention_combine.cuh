@@ -6,11 +6,13 @@ namespace fsie {
 
 // Merge the key splits of one (token, head); same arithmetic as attention_generic.cu.  The
 // weights e^(m_z - M) of splits z and z + 32 are computed once by lane z (nsplit <= 64) and
-// broadcast.
+// broadcast.  With `gate` (head h of token t at t * gate_ld + h * HD) the result is multiplied by its
+// sigmoid column by column before it is rounded.
 constexpr int MAX_KEY_SPLITS = 64;
 __global__ void attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                         bf16* __restrict__ out, int out_ld, int tokens, int heads,
-                                        int nsplit, const int* __restrict__ token_list) {
+                                        int nsplit, const int* __restrict__ token_list,
+                                        const bf16* __restrict__ gate, int gate_ld) {
     // the list of tokens was staged before the step: it is read while the attention kernel still runs
     const int tok = token_list ? token_list[blockIdx.x] : blockIdx.x, h = blockIdx.y;
     grid_dependency_wait();
@@ -67,9 +69,15 @@ __global__ void attn_combine_kernel(const float* __restrict__ part_o, const floa
                 if (z0 + j < nsplit && w != 0.f) { a0 += v[j].x * w; a1 += v[j].y * w; }   // a split without keys may hold anything
             }
         }
-        if (mine)
-            *reinterpret_cast<__nv_bfloat162*>(out + (size_t)tok * out_ld + h * HD + d) =
-                __floats2bfloat162_rn(a0 * inv, a1 * inv);
+        if (mine) {
+            a0 *= inv; a1 *= inv;
+            if (gate) {
+                const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gate + (size_t)tok * gate_ld + h * HD + d));
+                a0 *= 1.0f / (1.0f + expf(-z.x));
+                a1 *= 1.0f / (1.0f + expf(-z.y));
+            }
+            *reinterpret_cast<__nv_bfloat162*>(out + (size_t)tok * out_ld + h * HD + d) = __floats2bfloat162_rn(a0, a1);
+        }
     }
 }
 

@@ -25,6 +25,13 @@
 //                   range is split)
 //
 // Formula: src/model/nn.cpp:151-226 of the reference, as a running softmax.
+//
+// WIDE form (fsie_attn_tc_scaled), for attention whose weights stay 32-bit on their way to the values
+// and whose scores have a scale per head, a cap or chunks: the scores are brought to base-2 units as
+// soon as they are read (CAP: through cap * tanh(s / cap) first), P is written as two bfloat16 halves -
+// the weight, and what rounding it lost - over both halves of the S columns, and O takes both; a
+// query may be confined to the keys of its own chunk of positions, and the result may be multiplied by
+// the sigmoid of a gate column by column before it is rounded.
 // Every wait on an mbarrier is bounded; when one runs out *error is set, all roles leave their
 // loops, tensor memory is freed and the kernel returns.
 #include "common.cuh"
@@ -67,7 +74,13 @@ constexpr uint32_t TMEM_COLS = 512;     // S_A | S_B | O_A | O_B, 128 columns ea
 constexpr uint32_t COL_S = 0, COL_O = STREAMS * BN;
 enum { ERR_TC_PRODUCER = 31, ERR_TC_MMA = 32, ERR_TC_SOFTMAX = 33, ERR_TC_LAYOUT = 34 };
 
-struct TcExtra { int entries, entry; int* error; };
+struct TcExtra {
+    int entries, entry; int* error;
+    const float* head_scale;           // [heads], the WIDE form's scale (p.scale otherwise)
+    int chunk;                         // > 0: a query sees only the keys of its own chunk of this many positions
+    float softcap;                     // CAP: scores pass through softcap * tanh(s / softcap)
+    const bf16* gate; int gate_ld;     // null, or head h of token t at t * gate_ld + h * HD
+};
 #define TC_MARK(slot) do { } while (0)
 
 }  // namespace fsie
@@ -125,6 +138,13 @@ __device__ __forceinline__ void tmem_st32_issue(uint32_t taddr, const uint32_t* 
                    "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31])
                  : "memory");
 }
+__device__ __forceinline__ void tmem_st16_issue(uint32_t taddr, const uint32_t* r) {
+    asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], "
+                 "{%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};"
+                 ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]),
+                   "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
+                 : "memory");
+}
 __device__ __forceinline__ void tmem_ld32(uint32_t taddr, float (&v)[32]) {
     uint32_t r[32];
     asm volatile("tcgen05.ld.sync.aligned.32x32b.x32.b32 "
@@ -161,6 +181,13 @@ __device__ __forceinline__ float fast_exp2(float v) {
 // byte offset of 16-byte chunk `chunk` (0..7) of row `row` inside a 128-byte-swizzled block
 __device__ __forceinline__ int swizzled(int row, int chunk) { return row * 128 + ((chunk ^ (row & 7)) << 4); }
 
+__device__ __forceinline__ float fast_rcp(float v) {
+    float r;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+    return r;
+}
+
+template <bool WIDE, bool CAP>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_tc_kernel(const __grid_constant__ CUtensorMap pages_map, const AttnParams p, const TcExtra x) {
     extern __shared__ __align__(1024) unsigned char smem_all[];
@@ -190,6 +217,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap pages_map, const AttnParams p
     const int pos_first = pos0 + row0 / group;
     const int pos_last = pos0 + (row0 + nrows - 1) / group;
     int kbegin = p.window > 0 ? max(0, pos_first - p.window + 1) : 0;
+    if (WIDE && x.chunk > 0) kbegin = max(kbegin, pos_first - pos_first % x.chunk);
     // tiles hold whole pages, and keys before the window are masked: the range starts on a tile
     // boundary before it is split, so that the splits' ranges stay disjoint
     kbegin = kbegin / BN * BN;
@@ -338,6 +366,12 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap pages_map, const AttnParams p
                         mma_ts(tmem + COL_O + st * BN, tmem + COL_S + st * BN + k * 8, vd + (uint64_t)(k * (16 * 128 >> 4)),
                                idesc_o, (i > 0 || k > 0) ? 1u : 0u);
                     }
+                    if (WIDE) {                                 // what rounding the weights lost
+#pragma unroll
+                        for (int k = 0; k < BN / 16; ++k)
+                            mma_ts(tmem + COL_O + st * BN, tmem + COL_S + st * BN + BN / 2 + k * 8,
+                                   vd + (uint64_t)(k * (16 * 128 >> 4)), idesc_o, 1u);
+                    }
                     if (i + 1 == ntiles) mma_commit(&ctl.o_done[st]);       // O_st is complete
                     if (st == streams - 1) mma_commit(&ctl.ring_empty[(2 * i + 1) % SLOTS]);    // V_i may be overwritten
                     if (i + 1 < ntiles) {                       // the stream's next scores, while the other's softmax runs
@@ -357,8 +391,14 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap pages_map, const AttnParams p
         const uint32_t s_addr = lane_base + COL_S + st * BN, o_addr = lane_base + COL_O + st * BN;
         const bool valid = st * BM + r < nrows;
         const int pos = valid ? pos0 + (row0 + st * BM + r) / group : -1;
-        const int lowest = p.window > 0 ? pos - p.window : -1;       // keys <= this are unseen
-        const float sc = p.scale * 1.4426950408889634f;
+        int lowest = p.window > 0 ? pos - p.window : -1;             // keys <= this are unseen
+        if (WIDE && x.chunk > 0 && pos >= 0) lowest = max(lowest, pos - pos % x.chunk - 1);
+        constexpr float LOG2E = 1.4426950408889634f;
+        // WIDE: the scores are in base-2 units before anything is done with them
+        const float sc = WIDE ? 1.f : p.scale * LOG2E;
+        const float natural = WIDE ? x.head_scale[kvh * group + (row0 + (valid ? st * BM + r : 0)) % group] : 0.f;
+        const float to_base2 = CAP ? 2.f * LOG2E * natural / x.softcap : LOG2E * natural;
+        const float cap2 = CAP ? LOG2E * x.softcap : 0.f;
         float m_run = -INFINITY, l_run = 0.f;
         bool ok = true;
         for (int i = 0; i < ntiles && ok; ++i) {
@@ -377,6 +417,15 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap pages_map, const AttnParams p
             for (int c = 0; c < BN; c += 32) tmem_ld32_issue(s_addr + c, sr + c);
             tmem_wait_ld();
             TC_MARK(1);
+            if (WIDE) {
+#pragma unroll
+                for (int j = 0; j < BN; ++j) {
+                    float v = __uint_as_float(sr[j]) * to_base2;
+                    // cap * tanh(s / cap) with tanh(x) = 1 - 2 / (1 + e^(2 x)), times log2 e
+                    if (CAP) v = fmaf(-2.f * cap2, fast_rcp(1.f + fast_exp2(v)), cap2);
+                    sr[j] = __float_as_uint(v);
+                }
+            }
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};      // four chains, not one
             const bool clear = k0 + BN - 1 < kend && k0 + BN - 1 <= pos && k0 > lowest;   // nothing to mask
             if (__all_sync(0xffffffffu, clear || !valid)) {
@@ -420,17 +469,40 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap pages_map, const AttnParams p
             // p = exp2(s * sc - base), row sum, P as bfloat16 pairs (key 2 c low, key 2 c + 1 high in
             // column c) over the registers that held the scores
             float sum4[4] = {0.f, 0.f, 0.f, 0.f};
+            if (WIDE) {
+                // 32 keys at a time: 16 columns of weights, and 16 of what rounding them lost
 #pragma unroll
-            for (int j = 0; j < BN; j += 2) {
-                const float p0 = fast_exp2(fmaf(__uint_as_float(sr[j]), sc, -base));
-                const float p1 = fast_exp2(fmaf(__uint_as_float(sr[j + 1]), sc, -base));
-                sum4[(j >> 1) & 1] += p0;
-                sum4[2 + ((j >> 1) & 1)] += p1;
-                __nv_bfloat162 h2 = __floats2bfloat162_rn(p0, p1);
-                sr[j >> 1] = *reinterpret_cast<uint32_t*>(&h2);
+                for (int part = 0; part < 4; ++part) {
+                    uint32_t lost[16];
+#pragma unroll
+                    for (int c = 0; c < 16; ++c) {
+                        const int j = part * 32 + 2 * c;
+                        const float p0 = fast_exp2(__uint_as_float(sr[j]) - base);
+                        const float p1 = fast_exp2(__uint_as_float(sr[j + 1]) - base);
+                        sum4[c & 1] += p0;
+                        sum4[2 + (c & 1)] += p1;
+                        const __nv_bfloat162 hi = __floats2bfloat162_rn(p0, p1);
+                        const float2 back = __bfloat1622float2(hi);
+                        const __nv_bfloat162 lo = __floats2bfloat162_rn(p0 - back.x, p1 - back.y);
+                        sr[part * 16 + c] = *reinterpret_cast<const uint32_t*>(&hi);
+                        lost[c] = *reinterpret_cast<const uint32_t*>(&lo);
+                    }
+                    tmem_st16_issue(s_addr + part * 16, sr + part * 16);
+                    tmem_st16_issue(s_addr + BN / 2 + part * 16, lost);
+                }
+            } else {
+#pragma unroll
+                for (int j = 0; j < BN; j += 2) {
+                    const float p0 = fast_exp2(fmaf(__uint_as_float(sr[j]), sc, -base));
+                    const float p1 = fast_exp2(fmaf(__uint_as_float(sr[j + 1]), sc, -base));
+                    sum4[(j >> 1) & 1] += p0;
+                    sum4[2 + ((j >> 1) & 1)] += p1;
+                    __nv_bfloat162 h2 = __floats2bfloat162_rn(p0, p1);
+                    sr[j >> 1] = *reinterpret_cast<uint32_t*>(&h2);
+                }
+#pragma unroll
+                for (int c = 0; c < BN / 2; c += 32) tmem_st32_issue(s_addr + c, sr + c);
             }
-#pragma unroll
-            for (int c = 0; c < BN / 2; c += 32) tmem_st32_issue(s_addr + c, sr + c);
             tmem_wait_st();
             const float sum = valid ? (sum4[0] + sum4[1]) + (sum4[2] + sum4[3]) : 0.f;
             l_run = l_run * corr + sum;
@@ -464,6 +536,12 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap pages_map, const AttnParams p
 #pragma unroll
                 for (int g8 = 0; g8 < 4; ++g8) {
                     uint4 packed;
+                    if (WIDE && x.gate) {
+                        float z[8];
+                        load8(x.gate + (size_t)tok * x.gate_ld + h * HD + c + g8 * 8, z);
+#pragma unroll
+                        for (int j = 0; j < 8; ++j) v[g8 * 8 + j] *= 1.0f / (1.0f + expf(-z[j]));
+                    }
                     __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&packed);
 #pragma unroll
                     for (int j = 0; j < 4; ++j)
@@ -480,7 +558,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap pages_map, const AttnParams p
         }
         if (valid && p.nsplit > 1) {
             const size_t idx = ((size_t)split * p.tokens + tok) * p.heads + h;
-            p.part_ml[idx * 2] = m_run == -INFINITY ? -INFINITY : m_run * p.scale;
+            p.part_ml[idx * 2] = m_run == -INFINITY ? -INFINITY : m_run * (WIDE ? 0.6931471805599453f : p.scale);
             p.part_ml[idx * 2 + 1] = l_run;
         }
     }
@@ -549,13 +627,6 @@ __device__ __forceinline__ void tmem_ld16_issue(uint32_t taddr, uint32_t* r) {
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]),
                    "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
                  : "r"(taddr) : "memory");
-}
-__device__ __forceinline__ void tmem_st16_issue(uint32_t taddr, const uint32_t* r) {
-    asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], "
-                 "{%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};"
-                 ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]),
-                   "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
-                 : "memory");
 }
 // all 128 softmax threads meet; returns whether any of them brought `flag`
 __device__ __forceinline__ bool softmax_meet(bool flag) {
@@ -933,12 +1004,12 @@ int fsie_attn_tc_pages_map(void* map_out, const void* pages, long long total_row
 // Tiles of 256 query rows.  Arguments as fsie_attn_mma (attention_mma.cu) without a row class,
 // with the pages given as a TMA descriptor (`pages_map`, made by fsie_attn_tc_pages_map over
 // `entries` cache entries per page, of which this launch reads `entry`) and the error flag.
-int fsie_attn_tc(const void* pages_map, int entries, int entry, const void* q, int q_ld, int page_size,
+static int attn_tc_launch(const void* pages_map, int entries, int entry, const void* q, int q_ld, int page_size,
                  const int* block_tables, int bt_stride, const int* tile_item, const int* tile_row0, int tiles,
                  const int* item_qstart, const int* item_qlen, const int* item_pos0, void* out, int out_ld,
                  float* part_o, float* part_ml, int tokens, int heads, int kv_heads, int head_dim, int window,
-                 int nsplit, float scale, const int* combine_tokens, int num_combine, int* error,
-                 cudaStream_t stream) {
+                 int nsplit, float scale, const float* head_scale, int chunk, float softcap, const void* gate,
+                 int gate_ld, const int* combine_tokens, int num_combine, int* error, cudaStream_t stream) {
     if (tiles <= 0 || tokens <= 0) return 0;
     if (head_dim != HD) return ERR_UNSUPPORTED;
     if (page_size != 8 && page_size != 16 && page_size != 32 && page_size != 64 && page_size != 128) return ERR_UNSUPPORTED;
@@ -959,20 +1030,53 @@ int fsie_attn_tc(const void* pages_map, int entries, int entry, const void* q, i
     p.window = window; p.nsplit = nsplit; p.scale = scale;
     TcExtra x;
     x.entries = entries; x.entry = entry; x.error = error;
-    static bool configured = false;
-    if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attn_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES);
+    x.head_scale = head_scale; x.chunk = chunk; x.softcap = softcap; x.gate = (const bf16*)gate; x.gate_ld = gate_ld;
+    auto* kernel = !head_scale ? attn_tc_kernel<false, false>
+                               : (softcap > 0.f ? attn_tc_kernel<true, true> : attn_tc_kernel<true, false>);
+    const int form = !head_scale ? 0 : (softcap > 0.f ? 2 : 1);
+    static bool configured[3] = {false, false, false};
+    if (!configured[form]) {
+        cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES);
         if (e != cudaSuccess) return (int)e;
-        configured = true;
+        configured[form] = true;
     }
-    attn_tc_kernel<<<dim3(tiles * kv_heads, 1, nsplit), THREADS, SMEM_BYTES, stream>>>(map, p, x);
+    kernel<<<dim3(tiles * kv_heads, 1, nsplit), THREADS, SMEM_BYTES, stream>>>(map, p, x);
     int rc = (int)cudaGetLastError();
     if (rc != 0 || nsplit == 1) return rc;
     const int count = combine_tokens ? num_combine : tokens;
     if (count <= 0) return 0;
     attn_combine_kernel<<<dim3(count, heads), HD >= 128 ? 64 : 32, 0, stream>>>(
-        part_o, part_ml, (bf16*)out, out_ld, tokens, heads, nsplit, combine_tokens);
+        part_o, part_ml, (bf16*)out, out_ld, tokens, heads, nsplit, combine_tokens, (const bf16*)gate, gate_ld);
     return (int)cudaGetLastError();
+}
+
+int fsie_attn_tc(const void* pages_map, int entries, int entry, const void* q, int q_ld, int page_size,
+                 const int* block_tables, int bt_stride, const int* tile_item, const int* tile_row0, int tiles,
+                 const int* item_qstart, const int* item_qlen, const int* item_pos0, void* out, int out_ld,
+                 float* part_o, float* part_ml, int tokens, int heads, int kv_heads, int head_dim, int window,
+                 int nsplit, float scale, const int* combine_tokens, int num_combine, int* error,
+                 cudaStream_t stream) {
+    return attn_tc_launch(pages_map, entries, entry, q, q_ld, page_size, block_tables, bt_stride, tile_item, tile_row0,
+                          tiles, item_qstart, item_qlen, item_pos0, out, out_ld, part_o, part_ml, tokens, heads,
+                          kv_heads, head_dim, window, nsplit, scale, nullptr, 0, 0.f, nullptr, 0, combine_tokens,
+                          num_combine, error, stream);
+}
+
+// The WIDE form: weights as two bfloat16 halves, a scale per head (head_scale [heads], float), chunk > 0:
+// keys of the query's own chunk only, softcap > 0: capped scores, gate (null, or heads x head_dim columns
+// per token, rows gate_ld apart, on 16-byte borders): the result times its sigmoid.
+int fsie_attn_tc_scaled(const void* pages_map, int entries, int entry, const void* q, int q_ld, int page_size,
+                        const int* block_tables, int bt_stride, const int* tile_item, const int* tile_row0, int tiles,
+                        const int* item_qstart, const int* item_qlen, const int* item_pos0, void* out, int out_ld,
+                        float* part_o, float* part_ml, int tokens, int heads, int kv_heads, int head_dim, int window,
+                        int nsplit, const float* head_scale, int chunk, float softcap, const void* gate, int gate_ld,
+                        const int* combine_tokens, int num_combine, int* error, cudaStream_t stream) {
+    if (!head_scale || chunk < 0 || !(softcap >= 0.f) || (gate && (gate_ld % 8 || ((size_t)gate & 15))))
+        return ERR_BAD_ARGUMENT;
+    return attn_tc_launch(pages_map, entries, entry, q, q_ld, page_size, block_tables, bt_stride, tile_item, tile_row0,
+                          tiles, item_qstart, item_qlen, item_pos0, out, out_ld, part_o, part_ml, tokens, heads,
+                          kv_heads, head_dim, window, nsplit, 0.f, head_scale, chunk, softcap, gate, gate_ld,
+                          combine_tokens, num_combine, error, stream);
 }
 
 // Tiles of up to 16 query rows (decoded tokens, two-token portions): attn_tc_decode_kernel.
@@ -1018,7 +1122,7 @@ int fsie_attn_tc_decode(const void* pages_map, int entries, int entry, const voi
     if (count <= 0) return 0;
     return launch_dependent(attn_combine_kernel, dim3(count, heads), dim3(HD >= 128 ? 64 : 32), 0, stream,
                             (const float*)part_o, (const float*)part_ml, (bf16*)out, out_ld, tokens, heads, nsplit,
-                            combine_tokens);
+                            combine_tokens, (const bf16*)nullptr, 0);
 }
 #else
 int fsie_attn_tc_decode_rows() { return 0; }

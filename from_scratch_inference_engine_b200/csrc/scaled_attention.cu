@@ -790,8 +790,10 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
 template <typename T>
 __global__ void sa_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                   T* __restrict__ out, int out_ld, int tokens, int heads, int dv,
-                                  int nsplit, const T* __restrict__ gate, int gate_ld) {
-    const int tok = blockIdx.x, h = blockIdx.y;
+                                  int nsplit, const T* __restrict__ gate, int gate_ld,
+                                  const int* __restrict__ token_list) {
+    // the list of tokens was staged before the step: it is read while the attention kernel still runs
+    const int tok = token_list ? token_list[blockIdx.x] : blockIdx.x, h = blockIdx.y;
     grid_dependency_wait();
     grid_dependents_go();
     float mmax = -INFINITY;
@@ -1065,6 +1067,7 @@ int fsie_scaled_attention_tile_rows(int dtype, int key_dim, int value_dim, int v
 // With nsplit > 1 the caller gives part_o [nsplit, tokens, heads, value_dim] and part_ml
 // [nsplit, tokens, heads, 2] (float); the ranges are merged after the launch.  softcap 0: no cap on
 // the scores; gate null, or heads x value_dim columns per token of the storage type, rows gate_ld apart.
+// combine_tokens null: every token's ranges are merged, else those of the num_combine tokens it lists.
 int fsie_scaled_attention(const void* q, int q_ld, const float* head_scale, const void* k_pages,
                           const void* v_pages, long long page_stride, int page_size, int key_dim,
                           int value_dim, int values_in_keys, const int* block_tables, int bt_stride,
@@ -1072,7 +1075,8 @@ int fsie_scaled_attention(const void* q, int q_ld, const float* head_scale, cons
                           const int* item_qlen, const int* item_pos0, const int* item_slots, void* out,
                           int out_ld, float* part_o, float* part_ml, int tokens, int heads, int kv_heads,
                           int window, int chunk, float softcap, const void* gate, int gate_ld, int nsplit,
-                          int dtype, int form, int* error, cudaStream_t stream) {
+                          const int* combine_tokens, int num_combine, int dtype, int form, int* error,
+                          cudaStream_t stream) {
     if (tokens <= 0 || tiles <= 0) return 0;
     if (tiles > 65535 || nsplit > 65535) return ERR_UNSUPPORTED;
     if (key_dim <= 0 || value_dim <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || nsplit < 1 ||
@@ -1118,13 +1122,15 @@ int fsie_scaled_attention(const void* q, int q_ld, const float* head_scale, cons
                                 : scaled_attention_dispatch<bf16>(p, tiles, values_in_keys != 0, stream);
     }
     if (rc != 0 || nsplit == 1) return rc;
-    const dim3 cgrid(tokens, heads);
+    const dim3 cgrid(combine_tokens ? num_combine : tokens, heads);
+    if (cgrid.x == 0) return 0;
     const int threads = value_dim >= 128 ? 128 : (value_dim >= 64 ? 64 : 32);
     if (dtype == DTYPE_F32)
         return launch_dependent(sa_combine_kernel<float>, cgrid, dim3(threads), 0, stream, part_o, part_ml, (float*)out,
-                                out_ld, tokens, heads, value_dim, nsplit, (const float*)gate, gate_ld);
+                                out_ld, tokens, heads, value_dim, nsplit, (const float*)gate, gate_ld,
+                                combine_tokens);
     return launch_dependent(sa_combine_kernel<bf16>, cgrid, dim3(threads), 0, stream, part_o, part_ml, (bf16*)out,
-                            out_ld, tokens, heads, value_dim, nsplit, (const bf16*)gate, gate_ld);
+                            out_ld, tokens, heads, value_dim, nsplit, (const bf16*)gate, gate_ld, combine_tokens);
 }
 
 // proj [tokens, ld] = q | k | v head by head; cos_sin [table_len, rotary_dim]; slot_of [tokens]

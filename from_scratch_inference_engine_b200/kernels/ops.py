@@ -384,9 +384,11 @@ def attn_tc(head_dim: int):
         lib.fsie_attn_tc.argtypes = [p, i, i, p, i, i, p, i, p, p, i, p, p, p, p, i, p, p,
                                      i, i, i, i, i, i, f, p, i, p, p]
         lib.fsie_attn_tc_decode.argtypes = lib.fsie_attn_tc.argtypes
+        lib.fsie_attn_tc_scaled.argtypes = [p, i, i, p, i, i, p, i, p, p, i, p, p, p, p, i, p, p,
+                                            i, i, i, i, i, i, p, i, f, p, i, p, i, p, p]
         lib.fsie_attn_tc_decode_rows.argtypes = []
         for name in ("fsie_attn_tc_map_bytes", "fsie_attn_tc_pages_map", "fsie_attn_tc",
-                     "fsie_attn_tc_decode", "fsie_attn_tc_decode_rows"):
+                     "fsie_attn_tc_scaled", "fsie_attn_tc_decode", "fsie_attn_tc_decode_rows"):
             getattr(lib, name).restype = i
         _attn_tc[head_dim] = lib
     return _attn_tc[head_dim]
@@ -421,7 +423,7 @@ def attention_tc(pages_map: PagesMap, entry: int, q: torch.Tensor, q_ld: int,
                  part_o: Optional[torch.Tensor] = None, part_ml: Optional[torch.Tensor] = None,
                  combine_tokens: Optional[torch.Tensor] = None, num_combine: int = 0
                  ) -> torch.Tensor:
-    """bfloat16 attention of prompt portions (tiles of 128 query rows) with tcgen05.mma."""
+    """bfloat16 attention of prompt portions (tiles of 256 query rows) with tcgen05.mma."""
     for name, t in (("block_tables", block_tables), ("tile_item", tile_item),
                     ("tile_row0", tile_row0), ("item_qstart", item_qstart),
                     ("item_qlen", item_qlen), ("item_pos0", item_pos0), ("error", error)):
@@ -441,6 +443,41 @@ def attention_tc(pages_map: PagesMap, entry: int, q: torch.Tensor, q_ld: int,
         _ptr(item_qstart), _ptr(item_qlen), _ptr(item_pos0), _ptr(out), out.stride(0),
         _ptr(part_o), _ptr(part_ml), tokens, heads, kv_heads, head_dim, window, nsplit,
         float(scale), _ptr(combine_tokens), num_combine, _ptr(error), _stream()), "attention_tc")
+    return out
+
+
+def attention_tc_scaled(pages_map: PagesMap, entry: int, q: torch.Tensor, q_ld: int, head_scale: torch.Tensor,
+                        block_tables: torch.Tensor, tile_item: torch.Tensor, tile_row0: torch.Tensor,
+                        num_tiles: int, item_qstart: torch.Tensor, item_qlen: torch.Tensor,
+                        item_pos0: torch.Tensor, out: torch.Tensor, tokens: int, heads: int,
+                        kv_heads: int, window: int, error: torch.Tensor, nsplit: int = 1,
+                        part_o: Optional[torch.Tensor] = None, part_ml: Optional[torch.Tensor] = None,
+                        chunk: int = 0, softcap: float = 0.0, gate: Optional[torch.Tensor] = None,
+                        combine_tokens: Optional[torch.Tensor] = None, num_combine: int = 0) -> torch.Tensor:
+    """`scaled_attention` of prompt portions (bfloat16, keys and values as wide as `pages_map` says, tiles
+    of `ATTENTION_TC_ROWS` query rows) with tcgen05.mma; the weights meet the values as two bfloat16
+    halves.  `gate` rows and its first column start on 16 bytes."""
+    _need(q, torch.bfloat16, "q", contiguous=False)
+    _need(out, torch.bfloat16, "out")
+    _need(head_scale, torch.float32, "head_scale")
+    head_dim = pages_map.head_dim
+    if head_scale.numel() != heads or out.numel() < tokens * heads * head_dim:
+        raise KernelError("attention_tc_scaled: shapes do not fit")
+    gate_ld = 0
+    if gate is not None:
+        _need(gate, torch.bfloat16, "gate", contiguous=False)
+        if gate.shape != (tokens, heads * head_dim) or gate.stride(1) != 1:
+            raise KernelError("attention_tc_scaled: gate is not of the result's shape")
+        gate_ld = gate.stride(0)
+    if nsplit > 1 and (part_o.numel() < nsplit * tokens * heads * head_dim or
+                       part_ml.numel() < nsplit * tokens * heads * 2):
+        raise KernelError("attention_tc_scaled: split scratch is too small")
+    _check(attn_tc(head_dim).fsie_attn_tc_scaled(
+        pages_map.ptr, pages_map.entries, entry, _ptr(q), q_ld, pages_map.page_size, _ptr(block_tables),
+        block_tables.stride(0), _ptr(tile_item), _ptr(tile_row0), num_tiles, _ptr(item_qstart), _ptr(item_qlen),
+        _ptr(item_pos0), _ptr(out), heads * head_dim, _ptr(part_o), _ptr(part_ml), tokens, heads, kv_heads, head_dim,
+        window, nsplit, _ptr(head_scale), int(chunk), float(softcap), _ptr(gate), gate_ld, _ptr(combine_tokens),
+        num_combine, _ptr(error), _stream()), "attention_tc_scaled")
     return out
 
 
@@ -1300,7 +1337,7 @@ def mixers():
         lib.fsie_scaled_attention_tile_rows.argtypes = [i, i, i, i, i]
         lib.fsie_scaled_attention_tile_rows.restype = i
         lib.fsie_scaled_attention.argtypes = [p, i, p, p, p, ll, i, i, i, i, p, i, p, p, i, p, p, p, p,
-                                              p, i, p, p, i, i, i, i, i, f, p, i, i, i, i, p, p]
+                                              p, i, p, p, i, i, i, i, i, f, p, i, i, p, i, i, i, p, p]
         lib.fsie_norm_rotate_write.argtypes = [p, i, p, p, i, p, p, p, ll, i, i, i, i, i, i, i, p, p, f,
                                                i, i, p, p]
         lib.fsie_head_gate.argtypes = [p, i, p, i, i, i, i, i, p]
@@ -1414,15 +1451,17 @@ def scaled_attention(q: torch.Tensor, q_ld: int, head_scale: torch.Tensor, k_pag
                      kv_heads: int, window: int, error: torch.Tensor, nsplit: int = 1,
                      part_o: Optional[torch.Tensor] = None,
                      part_ml: Optional[torch.Tensor] = None, form: str = "auto",
-                     chunk: int = 0, softcap: float = 0.0,
-                     gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     chunk: int = 0, softcap: float = 0.0, gate: Optional[torch.Tensor] = None,
+                     combine_tokens: Optional[torch.Tensor] = None, num_combine: int = 0) -> torch.Tensor:
     """Causal (optionally windowed; `chunk` > 0: only over the keys j with j // chunk == i // chunk)
     softmax attention of q [tokens, heads x key_dim] over paged keys
     [kv_head][slot][key_dim] and values [kv_head][slot][value_dim] (or, values_in_keys, the first
     value_dim columns of the key rows), scores multiplied by head_scale[head] and - `softcap` > 0 -
     passed through softcap * tanh(. / softcap); scores, softmax and weights in 32-bit.  `gate`
     [tokens, heads x value_dim] (may be a view of columns of a wider tensor): the result is multiplied
-    by its sigmoid column by column before it is rounded.  `form`: "auto" takes a tensor-core kernel where one fits (bfloat16, key
+    by its sigmoid column by column before it is rounded.  `combine_tokens` (int32, `num_combine` of them): the tokens
+    that the tiles hold, where they are not all the step's tokens (split ranges of others are not
+    merged).  `form`: "auto" takes a tensor-core kernel where one fits (bfloat16, key
     sizes in steps of 16, value sizes 64 ... 512), "plain" the 32-bit kernel, "mma" insists on a
     tensor-core kernel, "mma_split" on the one whose warps split the value columns.  The tiles
     hold `scaled_attention_rows(dtype, key_dim, value_dim, values_in_keys, form)` rows."""
@@ -1448,7 +1487,7 @@ def scaled_attention(q: torch.Tensor, q_ld: int, head_scale: torch.Tensor, k_pag
         value_dim, int(values_in_keys), _ptr(block_tables), block_tables.stride(0), _ptr(tile_item),
         _ptr(tile_row0), tiles, _ptr(item_qstart), _ptr(item_qlen), _ptr(item_pos0), _ptr(item_slots),
         _ptr(out), heads * value_dim, _ptr(part_o), _ptr(part_ml), tokens, heads, kv_heads, window,
-        int(chunk), float(softcap), _ptr(gate), gate_ld, nsplit, _tag(q.dtype), SCALED_ATTENTION_FORMS[form], _ptr(error), _stream()),
+        int(chunk), float(softcap), _ptr(gate), gate_ld, nsplit, _ptr(combine_tokens), num_combine, _tag(q.dtype), SCALED_ATTENTION_FORMS[form], _ptr(error), _stream()),
         "scaled_attention")
     return out
 

@@ -11,11 +11,13 @@ from ..cache.manager import CacheNeed
 from ..config.spec import PartSpec
 from ..kernels import ops
 from ..weights.tensor_spec import TensorSpec
+from .attention import attention_splits
 from .base import LayerCache, Mixer, build_part, register_part
 
 MAX_KEY_SPLITS = 64
 # which form of the attention kernel `attend` asks for: "auto" (a tensor-core kernel where one takes
-# the sizes), or "plain" to measure or test the 32-bit kernel in its place
+# the sizes: tcgen05 for portions of many query rows, mma.sync for the others), "mma" for mma.sync
+# only, or "plain" to measure or test the 32-bit kernel in their place
 FORM = "auto"
 
 
@@ -32,10 +34,13 @@ def attend(ctx, rt, q: torch.Tensor, head_scale: torch.Tensor, group, cache: Lay
            out: torch.Tensor, heads: int, kv_heads: int, key_dim: int, value_dim: int,
            values_in_keys: bool, window: int, chunk: int = 0, softcap: float = 0.0,
            gate: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """The step's tokens over the pages through `ops.scaled_attention`: tiles of query rows, key
-    ranges split over blocks when the tiles are few."""
+    """The step's tokens over the pages: tiles of query rows, key ranges split over blocks when the
+    tiles are few.  In bfloat16 with keys and values of one width that the tcgen05 kernel takes,
+    requests that bring more query rows than one tile of `ops.scaled_attention` holds go to it, the
+    others (decoded tokens, short portions) to `ops.scaled_attention`; elsewhere all go to that."""
     tokens = q.shape[0]
-    form = FORM
+    # "mma": "auto" without the tcgen05 kernel (the entry point's own "mma" refuses what it cannot take)
+    form = "auto" if FORM == "mma" else FORM
     value_ld = key_dim if values_in_keys else value_dim
     if form == "auto" and (q.stride(0) % 8 or cache.page_stride % 8 or value_ld % 8 or q.data_ptr() % 16
                            or cache.k_pages.data_ptr() % 16 or cache.v_pages.data_ptr() % 16
@@ -43,22 +48,44 @@ def attend(ctx, rt, q: torch.Tensor, head_scale: torch.Tensor, group, cache: Lay
                            or (gate is not None and (gate.stride(0) % 2 or gate.data_ptr() % 4))):
         form = "plain"          # rows that do not start where the tensor-core kernels' 16-byte copies need them
     rows = ops.scaled_attention_rows(q.dtype, key_dim, value_dim, values_in_keys, form)
-    tiles = ctx.attention_tiles(heads // kv_heads, rows)
     reach = min(window if window > 0 else chunk, chunk if chunk > 0 else window)   # 0: every key
-    longest = ctx.max_context if reach <= 0 else min(ctx.max_context, reach + rows)
-    nsplit = key_splits(tiles.count * kv_heads, longest, rt.sm_count,
-                        key_tile=64 if q.dtype is torch.bfloat16 else 32)
-    part_o = part_ml = None
-    if nsplit > 1:
-        part_o = ctx.scratch("scaled_attention.part_o", nsplit * tokens * heads * value_dim)
-        part_ml = ctx.scratch("scaled_attention.part_ml", nsplit * tokens * heads * 2)
-    return ops.scaled_attention(q, q.stride(0), head_scale, cache.k_pages, cache.v_pages,
-                                cache.page_stride, group.page_size, key_dim, value_dim,
-                                values_in_keys, group.block_tables, tiles.item, tiles.row0,
-                                tiles.count, ctx.item_qstart, ctx.item_qlen, ctx.item_pos0,
-                                ctx.item_slots, out, tokens, heads, kv_heads, window, ctx.error,
-                                nsplit, part_o, part_ml, form=form, chunk=chunk, softcap=softcap,
-                                gate=gate)
+
+    def scratch(nsplit: int):
+        if nsplit <= 1:
+            return None, None
+        return (ctx.scratch("scaled_attention.part_o", nsplit * tokens * heads * value_dim),
+                ctx.scratch("scaled_attention.part_ml", nsplit * tokens * heads * 2))
+
+    pages_map = None
+    if FORM == "auto" and form == "auto" and q.dtype is torch.bfloat16 and cache.pages is not None \
+            and (gate is None or (gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0)):
+        pages_map = rt.pages_map(cache.pages)
+    if pages_map is None:
+        launches = [(0, ctx.attention_tiles(heads // kv_heads, rows), None, 0, ctx.max_context)]
+    else:
+        launches = ctx.attention_row_classes(heads // kv_heads, (rows, ops.ATTENTION_TC_ROWS))
+    for row_class, tiles, class_tokens, count, longest in launches:
+        if reach > 0:
+            longest = min(longest, reach + (ops.ATTENTION_TC_ROWS if row_class else rows))
+        if row_class:
+            nsplit = attention_splits(tiles.count * kv_heads, longest, rt.sm_count, False, blocks_per_sm=1)
+            ops.attention_tc_scaled(pages_map, cache.entry_index, q, q.stride(0), head_scale,
+                                    group.block_tables, tiles.item, tiles.row0, tiles.count,
+                                    ctx.item_qstart, ctx.item_qlen, ctx.item_pos0, out, tokens, heads,
+                                    kv_heads, window, ctx.error, nsplit, *scratch(nsplit), chunk=chunk,
+                                    softcap=softcap, gate=gate, combine_tokens=class_tokens,
+                                    num_combine=count)
+            continue
+        nsplit = key_splits(tiles.count * kv_heads, longest, rt.sm_count,
+                            key_tile=64 if q.dtype is torch.bfloat16 else 32)
+        ops.scaled_attention(q, q.stride(0), head_scale, cache.k_pages, cache.v_pages,
+                             cache.page_stride, group.page_size, key_dim, value_dim,
+                             values_in_keys, group.block_tables, tiles.item, tiles.row0,
+                             tiles.count, ctx.item_qstart, ctx.item_qlen, ctx.item_pos0,
+                             ctx.item_slots, out, tokens, heads, kv_heads, window, ctx.error,
+                             nsplit, *scratch(nsplit), form=form, chunk=chunk, softcap=softcap,
+                             gate=gate, combine_tokens=class_tokens, num_combine=count)
+    return out
 
 
 @register_part("mixer", "scaled_gqa_attention")

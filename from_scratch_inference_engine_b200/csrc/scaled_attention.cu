@@ -270,6 +270,8 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src, bool vali
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" :: "r"(smem_u32(dst)), "l"(src), "r"(bytes) : "memory");
 }
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int LEFT>                // all but the LEFT most recent groups have arrived
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" :: "n"(LEFT) : "memory"); }
 __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
 
 // two neighbouring columns of a result, times the sigmoid of their gates where there are any
@@ -544,29 +546,38 @@ __global__ void __launch_bounds__(SA_WARPS * 32) scaled_attention_mma_kernel(con
 // columns, so the weights never leave its registers (the score tile's accumulator layout is the
 // layout of the next product's first operand) and the warps of a block meet only where a tile of
 // keys changes hands.  A block is four warps = a tile of up to 64 query rows.
-constexpr int TR_ROWS = 64, TR_WARPS = 4;
+//
+// FEW: a tile of up to 16 query rows (decoded tokens).  All four warps own the same rows and each takes
+// 16 of a tile's 64 keys with maxima, sums and outputs of its own, so that no warp is without work;
+// they are merged through shared memory at the end.  Three slots: two tiles travel while one is
+// multiplied.
+constexpr int TR_ROWS = 64, TR_FEW_ROWS = 16, TR_WARPS = 4;
 
 struct RowsLayout {
     int ldk, ldv;
     size_t q_bytes, k_bytes, v_bytes, total;
-    __host__ __device__ RowsLayout(int dk, int dv, bool shared_v) {
+    __host__ __device__ RowsLayout(int dk, int dv, bool shared_v, bool few) {
+        const int slots = few ? 3 : 2;
         ldk = dk + TM_PAD; ldv = dv + TM_PAD;
-        q_bytes = (size_t)TR_ROWS * ldk * 2;
-        k_bytes = (size_t)2 * TM_KT * ldk * 2;
-        v_bytes = shared_v ? 0 : (size_t)2 * TM_KT * ldv * 2;
-        total = q_bytes + k_bytes + v_bytes + 2 * TM_KT * sizeof(int);
+        q_bytes = (size_t)(few ? TR_FEW_ROWS : TR_ROWS) * ldk * 2;
+        k_bytes = (size_t)slots * TM_KT * ldk * 2;      // FEW: at least 4 x 16 x dv floats for the merge
+        v_bytes = shared_v ? 0 : (size_t)slots * TM_KT * ldv * 2;
+        total = q_bytes + k_bytes + v_bytes;
     }
 };
 
-template <int NVT, bool SHARED_V>
+template <int NVT, bool SHARED_V, bool FEW>
 __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(const ScaledAttnParams p) {
     extern __shared__ __align__(16) unsigned char tr_smem[];
     const int dk = p.key_dim, dv = p.value_dim;
-    const RowsLayout L(dk, dv, SHARED_V);
-    bf16* Qs = reinterpret_cast<bf16*>(tr_smem);                                   // [64][ldk]
-    bf16* Ks = reinterpret_cast<bf16*>(tr_smem + L.q_bytes);                       // [2][64][ldk]
-    bf16* Vs = reinterpret_cast<bf16*>(tr_smem + L.q_bytes + L.k_bytes);           // [2][64][ldv]
-    int* key_ok = reinterpret_cast<int*>(tr_smem + L.q_bytes + L.k_bytes + L.v_bytes);   // [2][64]
+    constexpr int ROWS = FEW ? TR_FEW_ROWS : TR_ROWS;    // query rows of a tile
+    constexpr int WK = FEW ? TM_KT / TR_WARPS : TM_KT;   // keys of a tile that a warp takes
+    constexpr int SLOTS = FEW ? 3 : 2;
+    __shared__ float few_ml[FEW ? TR_WARPS : 1][TR_FEW_ROWS][2];
+    const RowsLayout L(dk, dv, SHARED_V, FEW);
+    bf16* Qs = reinterpret_cast<bf16*>(tr_smem);                                   // [ROWS][ldk]
+    bf16* Ks = reinterpret_cast<bf16*>(tr_smem + L.q_bytes);                       // [SLOTS][64][ldk]
+    bf16* Vs = reinterpret_cast<bf16*>(tr_smem + L.q_bytes + L.k_bytes);           // [SLOTS][64][ldv]
 
     // blocks start in the order of the grid: the last tiles of a prompt see the most keys and go first
     const int kvh = blockIdx.x, tile = gridDim.y - 1 - blockIdx.y, split = blockIdx.z;
@@ -577,10 +588,11 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
     if (p.item_slots && p.item_slots[item] < 0) return;
     const int row0 = p.tile_row0[tile];
     const int qstart = p.item_qstart[item], qlen = p.item_qlen[item], pos0 = p.item_pos0[item];
-    const int nrows = min(TR_ROWS, qlen * group - row0);
+    const int nrows = min(ROWS, qlen * group - row0);
     if (nrows <= 0) return;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int g = lane >> 2, t = lane & 3;
+    const int wrow = FEW ? 0 : warp * 16, wkey = FEW ? warp * WK : 0;    // this warp's first row and key of a tile
     const bf16* q = (const bf16*)p.q;
     const bf16* kp = (const bf16*)p.k_pages;
     const bf16* vp = (const bf16*)p.v_pages;
@@ -623,13 +635,22 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
             bf16* vdst = Vs + ((size_t)stage * TM_KT + j) * L.ldv;
             for (int c = part; c < dv / 8; c += TPR) cp_async16(vdst + c * 8, vsrc + c * 8, ok);
         }
-        if (part == 0) key_ok[stage * TM_KT + j] = ok;
         cp_async_commit();
     };
-    if (kbegin < kend) issue_tile(0, kbegin, page_of(kbegin));
-    int page_ahead = page_of(kbegin + TM_KT);
+    // every tile that could be asked for is a commit group of its own, an empty one beyond the range
+    {
+        int pages[SLOTS - 1];
+#pragma unroll
+        for (int s = 0; s < SLOTS - 1; ++s) pages[s] = page_of(kbegin + s * TM_KT);
+#pragma unroll
+        for (int s = 0; s < SLOTS - 1; ++s) {
+            if (kbegin + s * TM_KT < kend) issue_tile(s, kbegin + s * TM_KT, pages[s]);
+            else cp_async_commit();
+        }
+    }
+    int page_ahead = page_of(kbegin + (SLOTS - 1) * TM_KT);
 
-    for (int r = warp; r < TR_ROWS; r += TR_WARPS) {
+    for (int r = warp; r < ROWS; r += TR_WARPS) {
         const int row = row0 + r;
         const bf16* src = q + (size_t)(qstart + row / group) * p.q_ld + (size_t)(kvh * group + row % group) * dk;
         for (int c = lane; c < dk / 8; c += 32) {
@@ -643,44 +664,46 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
     float sc[2], m[2], l[2];
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
-        const int r = warp * 16 + g + 8 * i;
+        const int r = wrow + g + 8 * i;
         pos[i] = r < nrows ? pos0 + (row0 + r) / group : -1;
         first_key[i] = sa_first_key(p, pos[i]);
         sc[i] = r < nrows ? p.head_scale[kvh * group + (row0 + r) % group] : 0.f;
         m[i] = -INFINITY; l[i] = 0.f;
     }
     // the latest position among this warp's rows: tiles of keys beyond it are none of its business
-    const int warp_rows = min(16, nrows - warp * 16);
-    const int warp_last = warp_rows > 0 ? pos0 + (row0 + warp * 16 + warp_rows - 1) / group : -1;
-    const int warp_first = warp_rows > 0 ? pos0 + (row0 + warp * 16) / group : 0;
+    const int warp_rows = min(16, nrows - wrow);
+    const int warp_last = warp_rows > 0 ? pos0 + (row0 + wrow + warp_rows - 1) / group : -1;
+    const int warp_first = warp_rows > 0 ? pos0 + (row0 + wrow) / group : 0;
     const float cap_inv = p.softcap > 0.f ? 2.0f / p.softcap : 0.f;
     float acc[NVT][4];
 #pragma unroll
     for (int n = 0; n < NVT; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
     const int ldvv = SHARED_V ? L.ldk : L.ldv;
 
-    int it = 0;
-    for (int k0 = kbegin; k0 < kend; k0 += TM_KT, ++it) {
-        const int stage = it & 1;
-        cp_async_wait_all();
+    int stage = 0;
+    for (int k0 = kbegin; k0 < kend; k0 += TM_KT, stage = stage + 1 == SLOTS ? 0 : stage + 1) {
+        cp_async_wait<SLOTS - 2>();
         __syncthreads();                 // this tile has arrived; everybody is done with the tile before it
-        if (k0 + TM_KT < kend) {
-            issue_tile(stage ^ 1, k0 + TM_KT, page_ahead);
-            page_ahead = page_of(k0 + 2 * TM_KT);
+        if (k0 + (SLOTS - 1) * TM_KT < kend) {
+            issue_tile(stage == 0 ? SLOTS - 1 : stage - 1, k0 + (SLOTS - 1) * TM_KT, page_ahead);
+            page_ahead = page_of(k0 + SLOTS * TM_KT);
+        } else {
+            cp_async_commit();
         }
-        if (k0 > warp_last || k0 + TM_KT - 1 < sa_first_key(p, warp_first)) continue;
-        // ---- scores of 16 rows x 64 keys
-        float s[8][4];
+        if (k0 + wkey > warp_last || k0 + wkey + WK - 1 < sa_first_key(p, warp_first)) continue;
+        // ---- scores of 16 rows x WK keys
+        constexpr int NK = WK / 8;
+        float s[NK][4];
 #pragma unroll
-        for (int n = 0; n < 8; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+        for (int n = 0; n < NK; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
         {
-            const bf16* qa = Qs + (warp * 16 + (lane & 15)) * L.ldk + (lane >> 4) * 8;
-            const bf16* kb = Ks + ((size_t)stage * TM_KT + (lane & 7) + (lane >> 4) * 8) * L.ldk + ((lane >> 3) & 1) * 8;
+            const bf16* qa = Qs + (wrow + (lane & 15)) * L.ldk + (lane >> 4) * 8;
+            const bf16* kb = Ks + ((size_t)stage * TM_KT + wkey + (lane & 7) + (lane >> 4) * 8) * L.ldk + ((lane >> 3) & 1) * 8;
             for (int kk = 0; kk < dk; kk += 16) {
                 uint32_t a[4];
                 ldsm_x4(a, qa + kk);
 #pragma unroll
-                for (int nb = 0; nb < 4; ++nb) {
+                for (int nb = 0; nb < NK / 2; ++nb) {
                     uint32_t b[4];
                     ldsm_x4(b, kb + (size_t)nb * 16 * L.ldk + kk);
                     mma_bf16(s[2 * nb], a, b[0], b[1]);
@@ -690,22 +713,22 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
         }
         float tmax[2] = {-INFINITY, -INFINITY};
 #pragma unroll
-        for (int n = 0; n < 8; ++n)
+        for (int n = 0; n < NK; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) s[n][e] *= sc[e >> 1];
         if (p.softcap > 0.f) {
 #pragma unroll
-            for (int n = 0; n < 8; ++n)
+            for (int n = 0; n < NK; ++n)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) s[n][e] = sa_cap_fast(s[n][e], p.softcap, cap_inv);
         }
 #pragma unroll
-        for (int n = 0; n < 8; ++n)
+        for (int n = 0; n < NK; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int i = e >> 1;
                 const int j = n * 8 + 2 * t + (e & 1);
-                const int kj = k0 + j;
+                const int kj = k0 + wkey + j;
                 const bool seen = kj < kend && kj <= pos[i] && kj >= first_key[i];
                 if (!seen) s[n][e] = -INFINITY;
                 tmax[i] = fmaxf(tmax[i], s[n][e]);
@@ -721,7 +744,7 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
             l[i] *= corr[i];
         }
 #pragma unroll
-        for (int n = 0; n < 8; ++n)
+        for (int n = 0; n < NK; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 s[n][e] = s[n][e] == -INFINITY ? 0.f : __expf(s[n][e] - m[e >> 1]);
@@ -734,9 +757,9 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
         }
         // ---- 16 rows x all value columns += weights x values; the weights as two bfloat16 halves
         const bf16* vbase = (SHARED_V ? Ks + (size_t)stage * TM_KT * L.ldk : Vs + (size_t)stage * TM_KT * L.ldv) +
-                            ((lane & 7) + ((lane >> 3) & 1) * 8) * ldvv + (lane >> 4) * 8;
+                            (wkey + (lane & 7) + ((lane >> 3) & 1) * 8) * ldvv + (lane >> 4) * 8;
 #pragma unroll
-        for (int kk = 0; kk < 4; ++kk) {
+        for (int kk = 0; kk < WK / 16; ++kk) {
             uint32_t ah[4], al[4];
 #pragma unroll
             for (int x = 0; x < 4; ++x) {
@@ -759,11 +782,56 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
         }
     }
 
+    if (FEW) {
+        // the four warps' sums over their keys, merged: row r, columns d of every warp in shared memory,
+        // where the tiles were
+        __syncthreads();
+        float* merge = reinterpret_cast<float*>(tr_smem + L.q_bytes);               // [4][16][dv]
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            l[i] += __shfl_xor_sync(0xffffffffu, l[i], 1);
+            l[i] += __shfl_xor_sync(0xffffffffu, l[i], 2);
+            if (t == 0) { few_ml[warp][g + 8 * i][0] = m[i]; few_ml[warp][g + 8 * i][1] = l[i]; }
+            float* mine = merge + ((size_t)warp * TR_FEW_ROWS + g + 8 * i) * dv + 2 * t;
+#pragma unroll
+            for (int n = 0; n < NVT; ++n)
+                *reinterpret_cast<float2*>(mine + n * 8) = make_float2(acc[n][2 * i], acc[n][2 * i + 1]);
+        }
+        __syncthreads();
+        for (int e = tid; e < nrows * (NVT * 4); e += TR_WARPS * 32) {               // two columns each
+            const int r = e / (NVT * 4), d = (e - r * (NVT * 4)) * 2;
+            float mmax = -INFINITY;
+#pragma unroll
+            for (int w = 0; w < TR_WARPS; ++w) mmax = fmaxf(mmax, few_ml[w][r][0]);
+            float total = 0.f, a = 0.f, b = 0.f;
+#pragma unroll
+            for (int w = 0; w < TR_WARPS; ++w) {
+                const float f = few_ml[w][r][0] == -INFINITY ? 0.f : __expf(few_ml[w][r][0] - mmax);
+                const float2 v = *reinterpret_cast<const float2*>(merge + ((size_t)w * TR_FEW_ROWS + r) * dv + d);
+                total += f * few_ml[w][r][1];
+                a += f * v.x;
+                b += f * v.y;
+            }
+            const int row = row0 + r;
+            const int tok = qstart + row / group, h = kvh * group + row % group;
+            if (p.nsplit == 1) {
+                const float inv = total > 0.f ? 1.0f / total : 0.f;
+                const bf16* gate = p.gate ? (const bf16*)p.gate + (size_t)tok * p.gate_ld + (size_t)h * dv + d : nullptr;
+                *reinterpret_cast<__nv_bfloat162*>((bf16*)p.out + (size_t)tok * p.out_ld + (size_t)h * dv + d) =
+                    sa_gated_pair(a * inv, b * inv, gate);
+            } else {
+                const size_t idx = ((size_t)split * p.tokens + tok) * p.heads + h;
+                *reinterpret_cast<float2*>(p.part_o + idx * dv + d) = make_float2(a, b);
+                if (d == 0) { p.part_ml[idx * 2] = mmax; p.part_ml[idx * 2 + 1] = total; }
+            }
+        }
+        return;
+    }
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
         l[i] += __shfl_xor_sync(0xffffffffu, l[i], 1);
         l[i] += __shfl_xor_sync(0xffffffffu, l[i], 2);
-        const int r = warp * 16 + g + 8 * i;
+        const int r = wrow + g + 8 * i;
         if (r >= nrows) continue;
         const int row = row0 + r;
         const int tok = qstart + row / group, h = kvh * group + row % group;
@@ -786,7 +854,9 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
     }
 }
 
-// o = sum_z acc_z e^(m_z - M) / sum_z l_z e^(m_z - M) over the key ranges z of one (token, head)
+// o = sum_z acc_z e^(m_z - M) / sum_z l_z e^(m_z - M) over the key ranges z of one (token, head).  The
+// weights of 32 ranges at a time are worked out by the lanes of every warp and handed round by shuffles;
+// a range's values are asked for eight ranges at a time.
 template <typename T>
 __global__ void sa_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                   T* __restrict__ out, int out_ld, int tokens, int heads, int dv,
@@ -794,26 +864,44 @@ __global__ void sa_combine_kernel(const float* __restrict__ part_o, const float*
                                   const int* __restrict__ token_list) {
     // the list of tokens was staged before the step: it is read while the attention kernel still runs
     const int tok = token_list ? token_list[blockIdx.x] : blockIdx.x, h = blockIdx.y;
+    const int lane = threadIdx.x & 31;
+    const size_t stride = (size_t)tokens * heads, slot = (size_t)tok * heads + h;
     grid_dependency_wait();
     grid_dependents_go();
-    float mmax = -INFINITY;
-    for (int z = 0; z < nsplit; ++z)
-        mmax = fmaxf(mmax, part_ml[(((size_t)z * tokens + tok) * heads + h) * 2]);
-    float denom = 0.f;
-    for (int z = 0; z < nsplit; ++z) {
-        const size_t idx = ((size_t)z * tokens + tok) * heads + h;
-        const float mz = part_ml[idx * 2];
-        if (mz != -INFINITY) denom += part_ml[idx * 2 + 1] * expf(mz - mmax);
-    }
-    const float inv = denom > 0.f ? 1.0f / denom : 0.f;
-    for (int d = threadIdx.x; d < dv; d += blockDim.x) {
-        float o = 0.f;
-        for (int z = 0; z < nsplit; ++z) {
-            const size_t idx = ((size_t)z * tokens + tok) * heads + h;
-            const float mz = part_ml[idx * 2];
-            if (mz != -INFINITY) o += part_o[idx * dv + d] * expf(mz - mmax);
+    // every thread of a warp takes every turn of the loops (the weights travel by shuffles)
+    for (int d0 = 0; d0 < dv; d0 += blockDim.x) {
+        const int d = d0 + threadIdx.x;
+        const bool mine = d < dv;
+        float mmax = -INFINITY, denom = 0.f, o = 0.f;
+        for (int z0 = 0; z0 < nsplit; z0 += 32) {
+            const int zl = z0 + lane;
+            float mz = -INFINITY, lz = 0.f;
+            if (zl < nsplit) {
+                const float2 ml = *reinterpret_cast<const float2*>(part_ml + ((size_t)zl * stride + slot) * 2);
+                mz = ml.x;
+                lz = ml.y;
+            }
+            const float m_new = fmaxf(mmax, warp_max(mz));
+            const float corr = mmax == -INFINITY ? 0.f : expf(mmax - m_new);
+            const float w = mz == -INFINITY ? 0.f : expf(mz - m_new);
+            mmax = m_new;
+            denom = denom * corr + warp_sum(lz * w);
+            o *= corr;
+            const int n = min(32, nsplit - z0);
+            for (int j0 = 0; j0 < n; j0 += 8) {
+                float v[8];
+#pragma unroll
+                for (int j = 0; j < 8; ++j)
+                    v[j] = mine ? part_o[((size_t)(z0 + min(j0 + j, n - 1)) * stride + slot) * dv + d] : 0.f;
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    const float wj = __shfl_sync(0xffffffffu, w, min(j0 + j, 31));
+                    if (j0 + j < n && wj != 0.f) o += v[j] * wj;        // a range without keys may hold anything
+                }
+            }
         }
-        o *= inv;
+        if (!mine) continue;
+        o *= denom > 0.f ? 1.0f / denom : 0.f;
         if (gate) o *= sa_sigmoid(to_float(gate[(size_t)tok * gate_ld + (size_t)h * dv + d]));
         out[(size_t)tok * out_ld + (size_t)h * dv + d] = from_float<T>(o);
     }
@@ -1015,21 +1103,28 @@ static int scaled_attention_mma_launch(const ScaledAttnParams& p, int tiles, boo
     return launch_dependent(scaled_attention_mma_kernel<NV, false>, grid, dim3(SA_WARPS * 32), smem, stream, p);
 }
 
-template <int NVT>
+template <int NVT, bool FEW>
 static int scaled_attention_rows_launch(const ScaledAttnParams& p, int tiles, bool shared_v, cudaStream_t stream) {
-    const size_t smem = RowsLayout(p.key_dim, p.value_dim, shared_v).total;
+    const size_t smem = RowsLayout(p.key_dim, p.value_dim, shared_v, FEW).total;
     const dim3 grid(p.kv_heads, tiles, p.nsplit);
-    if (shared_v) {
-        cudaFuncSetAttribute(scaled_attention_rows_kernel<NVT, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        return launch_dependent(scaled_attention_rows_kernel<NVT, true>, grid, dim3(TR_WARPS * 32), smem, stream, p);
+    auto* kernel = shared_v ? scaled_attention_rows_kernel<NVT, true, FEW> : scaled_attention_rows_kernel<NVT, false, FEW>;
+    cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    return launch_dependent(kernel, grid, dim3(TR_WARPS * 32), smem, stream, p);
+}
+
+template <bool FEW>
+static int scaled_attention_rows_dispatch(const ScaledAttnParams& p, int tiles, bool shared_v, cudaStream_t stream) {
+    switch (p.value_dim / 64) {
+        case 1: return scaled_attention_rows_launch<8, FEW>(p, tiles, shared_v, stream);
+        case 2: return scaled_attention_rows_launch<16, FEW>(p, tiles, shared_v, stream);
+        case 3: return scaled_attention_rows_launch<24, FEW>(p, tiles, shared_v, stream);
+        default: return scaled_attention_rows_launch<32, FEW>(p, tiles, shared_v, stream);
     }
-    cudaFuncSetAttribute(scaled_attention_rows_kernel<NVT, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    return launch_dependent(scaled_attention_rows_kernel<NVT, false>, grid, dim3(TR_WARPS * 32), smem, stream, p);
 }
 
 // whether the tensor-core form of a warp per 16 rows takes these sizes (value sizes up to 256)
-static bool scaled_attention_rows_takes(int key_dim, int value_dim, bool shared_v) {
-    return value_dim <= 256 && RowsLayout(key_dim, value_dim, shared_v).total <= 227 * 1024;
+static bool scaled_attention_rows_takes(int key_dim, int value_dim, bool shared_v, bool few) {
+    return value_dim <= 256 && RowsLayout(key_dim, value_dim, shared_v, few).total <= 226 * 1024;
 }
 
 // whether the tensor-core form takes these sizes and addresses
@@ -1054,16 +1149,20 @@ int fsie_scaled_attention_rows() { return SA_ROWS; }
 // Query rows of one tile for these sizes: 64 where a warp of the tensor-core kernel owns 16 rows
 // with all their value columns (bfloat16, key sizes in steps of 16, value sizes 64, 128, 192, 256;
 // form 0 or 2), else 32.  The caller cuts its tile list accordingly.  form 3 asks for the
-// tensor-core kernel whose warps split the value columns at any value size it takes.
+// tensor-core kernel whose warps split the value columns at any value size it takes, form 4 for the one
+// whose warps split the keys of a tile of up to 16 rows (16, or 0 where it does not take the sizes).
 int fsie_scaled_attention_tile_rows(int dtype, int key_dim, int value_dim, int values_in_keys, int form) {
-    if (dtype != DTYPE_BF16 || form == 1 || form == 3 || key_dim % 16 || value_dim % 64) return SA_ROWS;
-    return scaled_attention_rows_takes(key_dim, value_dim, values_in_keys != 0) ? TR_ROWS : SA_ROWS;
+    const bool sizes = dtype == DTYPE_BF16 && key_dim % 16 == 0 && value_dim % 64 == 0;
+    if (form == 4)
+        return sizes && scaled_attention_rows_takes(key_dim, value_dim, values_in_keys != 0, true) ? TR_FEW_ROWS : 0;
+    if (!sizes || form == 1 || form == 3) return SA_ROWS;
+    return scaled_attention_rows_takes(key_dim, value_dim, values_in_keys != 0, false) ? TR_ROWS : SA_ROWS;
 }
 
 // values_in_keys != 0: v_pages is ignored, a key row's first value_dim columns are its value row.
 // form 0: the tensor-core kernel where it takes the sizes (bfloat16), else the 32-bit one; 1: the
 // 32-bit kernel; 2: a tensor-core kernel or refusal; 3: the tensor-core kernel whose warps split the
-// value columns, or refusal.  The tiles hold fsie_scaled_attention_tile_rows(...) rows.
+// value columns, or refusal; 4: the one whose warps split the keys, or refusal.  The tiles hold fsie_scaled_attention_tile_rows(...) rows.
 // With nsplit > 1 the caller gives part_o [nsplit, tokens, heads, value_dim] and part_ml
 // [nsplit, tokens, heads, 2] (float); the ranges are merged after the launch.  softcap 0: no cap on
 // the scores; gate null, or heads x value_dim columns per token of the storage type, rows gate_ld apart.
@@ -1097,15 +1196,12 @@ int fsie_scaled_attention(const void* q, int q_ld, const float* head_scale, cons
     p.error = error;
     int rc;
     const int tile_rows = fsie_scaled_attention_tile_rows(dtype, key_dim, value_dim, values_in_keys, form);
-    if (tile_rows == TR_ROWS) {
-        // the caller has cut tiles of 64 rows: no other kernel may take them
+    if (tile_rows == 0) return ERR_UNSUPPORTED;
+    if (tile_rows != SA_ROWS) {
+        // the caller has cut tiles of 64 (or 16) rows: no other kernel may take them
         if (!scaled_attention_mma_takes(p, dtype, values_in_keys != 0)) return ERR_UNSUPPORTED;
-        switch (value_dim / 64) {
-            case 1: rc = scaled_attention_rows_launch<8>(p, tiles, values_in_keys != 0, stream); break;
-            case 2: rc = scaled_attention_rows_launch<16>(p, tiles, values_in_keys != 0, stream); break;
-            case 3: rc = scaled_attention_rows_launch<24>(p, tiles, values_in_keys != 0, stream); break;
-            default: rc = scaled_attention_rows_launch<32>(p, tiles, values_in_keys != 0, stream); break;
-        }
+        rc = tile_rows == TR_ROWS ? scaled_attention_rows_dispatch<false>(p, tiles, values_in_keys != 0, stream)
+                                  : scaled_attention_rows_dispatch<true>(p, tiles, values_in_keys != 0, stream);
     } else if (form != 1 && scaled_attention_mma_takes(p, dtype, values_in_keys != 0)) {
         switch (value_dim / 32) {
             case 2: rc = scaled_attention_mma_launch<2>(p, tiles, values_in_keys != 0, stream); break;

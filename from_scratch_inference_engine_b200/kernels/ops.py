@@ -1429,13 +1429,14 @@ def mingru_scan(proj: torch.Tensor, width: int, item_qstart: torch.Tensor, item_
     return out
 
 
-SCALED_ATTENTION_FORMS = {"auto": 0, "plain": 1, "mma": 2, "mma_split": 3}
+SCALED_ATTENTION_FORMS = {"auto": 0, "plain": 1, "mma": 2, "mma_split": 3, "mma_few": 4}
 
 
 def scaled_attention_rows(dtype: torch.dtype = torch.float32, key_dim: int = 0, value_dim: int = 0,
                           values_in_keys: bool = False, form: str = "auto") -> int:
     """Query rows of one tile of `scaled_attention` for these sizes and this form of the kernel
-    (64 where a warp of the tensor-core kernel owns 16 rows with all their value columns, else 32)."""
+    (64 where a warp of the tensor-core kernel owns 16 rows with all their value columns, else 32;
+    "mma_few": 16, or 0 where that form does not take the sizes)."""
     if key_dim <= 0:
         return int(mixers().fsie_scaled_attention_rows())
     return int(mixers().fsie_scaled_attention_tile_rows(_tag(dtype), key_dim, value_dim,
@@ -1463,7 +1464,8 @@ def scaled_attention(q: torch.Tensor, q_ld: int, head_scale: torch.Tensor, k_pag
     that the tiles hold, where they are not all the step's tokens (split ranges of others are not
     merged).  `form`: "auto" takes a tensor-core kernel where one fits (bfloat16, key
     sizes in steps of 16, value sizes 64 ... 512), "plain" the 32-bit kernel, "mma" insists on a
-    tensor-core kernel, "mma_split" on the one whose warps split the value columns.  The tiles
+    tensor-core kernel, "mma_split" on the one whose warps split the value columns, "mma_few" on
+    the one for tiles of up to 16 rows whose warps split a tile's keys.  The tiles
     hold `scaled_attention_rows(dtype, key_dim, value_dim, values_in_keys, form)` rows."""
     _need(q, None, "q", contiguous=False)
     _need(head_scale, torch.float32, "head_scale")

@@ -36,8 +36,9 @@ def attend(ctx, rt, q: torch.Tensor, head_scale: torch.Tensor, group, cache: Lay
            gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The step's tokens over the pages: tiles of query rows, key ranges split over blocks when the
     tiles are few.  In bfloat16 with keys and values of one width that the tcgen05 kernel takes,
-    requests that bring more query rows than one tile of `ops.scaled_attention` holds go to it, the
-    others (decoded tokens, short portions) to `ops.scaled_attention`; elsewhere all go to that."""
+    requests that bring more query rows than one tile of `ops.scaled_attention` holds go to it; the
+    others, and all where it does not take the sizes, go to `ops.scaled_attention`: requests of few query
+    rows (decoded tokens) to its form for those, where there is one, the others to its form for many."""
     tokens = q.shape[0]
     # "mma": "auto" without the tcgen05 kernel (the entry point's own "mma" refuses what it cannot take)
     form = "auto" if FORM == "mma" else FORM
@@ -60,14 +61,23 @@ def attend(ctx, rt, q: torch.Tensor, head_scale: torch.Tensor, group, cache: Lay
     if FORM == "auto" and form == "auto" and q.dtype is torch.bfloat16 and cache.pages is not None \
             and (gate is None or (gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0)):
         pages_map = rt.pages_map(cache.pages)
-    if pages_map is None:
+    # (form, rows of its tiles) from few query rows to many; a request goes to the first whose tile
+    # holds all its rows, or to the last
+    classes = [(form, rows)]
+    few = ops.scaled_attention_rows(q.dtype, key_dim, value_dim, values_in_keys, "mma_few") if form == "auto" else 0
+    if few:
+        classes.insert(0, ("mma_few", few))
+    if pages_map is not None:
+        classes.append(("tcgen05", ops.ATTENTION_TC_ROWS))
+    if len(classes) == 1:
         launches = [(0, ctx.attention_tiles(heads // kv_heads, rows), None, 0, ctx.max_context)]
     else:
-        launches = ctx.attention_row_classes(heads // kv_heads, (rows, ops.ATTENTION_TC_ROWS))
+        launches = ctx.attention_row_classes(heads // kv_heads, tuple(r for _, r in classes))
     for row_class, tiles, class_tokens, count, longest in launches:
+        class_form, class_rows = classes[row_class]
         if reach > 0:
-            longest = min(longest, reach + (ops.ATTENTION_TC_ROWS if row_class else rows))
-        if row_class:
+            longest = min(longest, reach + class_rows)
+        if class_form == "tcgen05":
             nsplit = attention_splits(tiles.count * kv_heads, longest, rt.sm_count, False, blocks_per_sm=1)
             ops.attention_tc_scaled(pages_map, cache.entry_index, q, q.stride(0), head_scale,
                                     group.block_tables, tiles.item, tiles.row0, tiles.count,
@@ -83,7 +93,7 @@ def attend(ctx, rt, q: torch.Tensor, head_scale: torch.Tensor, group, cache: Lay
                              values_in_keys, group.block_tables, tiles.item, tiles.row0,
                              tiles.count, ctx.item_qstart, ctx.item_qlen, ctx.item_pos0,
                              ctx.item_slots, out, tokens, heads, kv_heads, window, ctx.error,
-                             nsplit, *scratch(nsplit), form=form, chunk=chunk, softcap=softcap,
+                             nsplit, *scratch(nsplit), form=class_form, chunk=chunk, softcap=softcap,
                              gate=gate, combine_tokens=class_tokens, num_combine=count)
     return out
 

@@ -294,7 +294,7 @@ def test_capped_scores_chunks_and_gated_columns(dtype, dk, dv, kv_heads, chunk, 
                      gated, seed=dk + chunk)
     forms = ["plain"]
     if dtype is torch.bfloat16 and dv % 64 == 0 and dk % 16 == 0:
-        forms += ["mma", "mma_split"] + (["tcgen05"] if dk == dv else [])
+        forms += ["mma", "mma_split", "mma_few"] + (["tcgen05"] if dk == dv else [])
     for form in forms:
         for nsplit in (1, 3):
             got, _ = case.run(form, nsplit)
@@ -325,7 +325,7 @@ def test_split_ranges_of_listed_tokens_only():
     stay as they were (another launch of the step fills them)."""
     case = Attention([(90, 200), (333, 1), (0, 150), (251, 1)], 4, 2, 64, 64, 16, torch.bfloat16, [0.4] * 4, 120, 0, 9.0,
                      True, seed=5)
-    for form, only in (("tcgen05", (0, 2)), ("auto", (1, 3)), ("plain", (1, 3))):
+    for form, only in (("tcgen05", (0, 2)), ("auto", (1, 3)), ("plain", (1, 3)), ("mma_few", (1, 3))):
         got, toks = case.run(form, 3, only)
         assert (got[toks] - case.want[toks]).abs().max() < 2e-2 * max(1.0, float(case.want.abs().max()))
         rest = torch.ones(case.tokens, dtype=torch.bool)

@@ -175,7 +175,8 @@ __global__ void stream_norm_kernel(const StreamNormParams p) {
 template <typename T, int S, int STEP>
 static int stream_norm_launch(const StreamNormParams& p, int num_rows, cudaStream_t stream) {
     const int columns = (p.width + STEP - 1) / STEP;
-    const int threads = S == 0 ? 128 : (columns >= 1024 ? 512 : (columns >= 256 ? 256 : 128));
+    // few rows: as many threads as there is work for, so that a row is one trip to memory
+    const int threads = S == 0 ? 128 : (columns >= (num_rows <= 64 ? 512 : 1024) ? 512 : (columns >= 256 ? 256 : 128));
     const size_t floats = (size_t)((p.width + 3) & ~3) + (size_t)p.streams * p.streams + 2 * (size_t)p.streams +
                           (S == 0 ? (size_t)p.streams * threads : 0);
     const size_t smem = floats * sizeof(float);

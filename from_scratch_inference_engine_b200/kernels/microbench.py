@@ -6,7 +6,10 @@ KERNEL: attention_decode, attention_prefill, add_rmsnorm, rope_kv_write, swiglu,
 sample, linear (the library product as the engine calls it), gemm_f32, gemm_decode,
 gemm_decode_swiglu, gemm_tiles, gemm_tiles_swiglu (the engine's own tcgen05 products),
 sum_layernorm, routed_experts (every kernel of a feed-forward of routed experts, one line for all),
-state_space (every kernel of a state-space mixer, and the same scan with one decay per head beside it).
+state_space (every kernel of a state-space mixer, and the same scan with one decay per head beside it),
+stream_norm (a residual of --streams streams settled, gathered and normed), scaled_attention (capped scores
+inside chunks of --chunk positions, gated columns: a prompt of --tokens behind --context - --tokens cached
+ones on tcgen05, or - --tokens 1 - decoded tokens of --batch requests on mma.sync; all flops are useful ones).
 
 Each kernel is timed with CUDA events over --iters launches after --warmup launches; between
 launches a buffer larger than L2 is read so that inputs come from HBM (read, not written:
@@ -166,6 +169,48 @@ def run_attention(args, timer, decode: bool):
                   "variant": ("tc" if use_tc else "tc_decode" if use_tcd else "mma")
                   if row_class >= 0 else ("rows16" if rows16 else "generic")})
     return ms, io_bytes, flops, extra
+
+
+def run_scaled_attention(args, timer):
+    """Attention with 32-bit weights, --softcap (0: none), chunks and a gate per column over shuffled pages."""
+    from ..parts.attention import attention_splits
+    from ..parts.scaled_attention import key_splits
+    heads, kv_heads, hd, page, new = args.heads, args.kv_heads, args.head_dim, args.page, args.tokens
+    batch, past, chunk = args.batch if new == 1 else 1, args.context - new, args.chunk
+    pages, tables, _, qstart, qlen, pos0 = paged_inputs(batch, new, past, heads, kv_heads, hd, page, torch.bfloat16)
+    group, tokens = heads // kv_heads, batch * new
+    wide = torch.randn(tokens, 2 * heads * hd, device="cuda").bfloat16()         # queries beside their gates
+    gate = wide[:, heads * hd:] if args.gate else None
+    scale = torch.full((heads,), hd ** -0.5, device="cuda")
+    out = torch.empty(tokens, heads * hd, dtype=torch.bfloat16, device="cuda")
+    error = torch.zeros(1, dtype=torch.int32, device="cuda")
+    sms = torch.cuda.get_device_properties(0).multi_processor_count
+    per_tile = 16 if new == 1 else ops.ATTENTION_TC_ROWS
+    tiles = [(i, r) for i in range(batch) for r in range(0, new * group, per_tile)]
+    tiles.sort(key=lambda t: -t[1])
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")
+    item, row0 = i32([t[0] for t in tiles]), i32([t[1] for t in tiles])
+    seen = lambda pos: pos % chunk + 1 if chunk else pos + 1
+    longest = min(args.context, chunk + per_tile) if chunk else args.context
+    nsplit = args.nsplit or (key_splits(len(tiles) * kv_heads, longest, sms, key_tile=64) if new == 1 else
+                             attention_splits(len(tiles) * kv_heads, longest, sms, False, blocks_per_sm=1))
+    parts = (torch.empty(nsplit * tokens * heads * hd, device="cuda"), torch.empty(nsplit * tokens * heads * 2, device="cuda"))
+    options = dict(chunk=chunk, softcap=args.softcap, gate=gate)
+    if new == 1:
+        slots = i32(list(range(batch)))
+        ms = timer(lambda: ops.scaled_attention(wide, wide.stride(0), scale, pages[:, 0, 0], pages[:, 0, 1], pages.stride(0),
+                                                page, hd, hd, False, tables, item, row0, len(tiles), qstart, qlen, pos0,
+                                                slots, out, tokens, heads, kv_heads, 0, error, nsplit, *parts,
+                                                form="mma_few", **options))
+    else:
+        pages_map = ops.PagesMap(pages, "tc")
+        ms = timer(lambda: ops.attention_tc_scaled(pages_map, 0, wide, wide.stride(0), scale, tables, item, row0, len(tiles),
+                                                   qstart, qlen, pos0, out, tokens, heads, kv_heads, 0, error, nsplit,
+                                                   *parts, **options))
+    keys = sum(seen(past + t) for t in range(new))
+    read = batch * min(args.context, seen(args.context - 1) if new == 1 else args.context)
+    nbytes = 2 * (read * 2 * kv_heads * hd + tokens * heads * hd * (3 if args.gate else 2))
+    return ms, nbytes, 4.0 * heads * hd * batch * keys, {"nsplit": nsplit, "tiles": len(tiles), "error": int(error.item())}
 
 
 def run_routed_experts(args, timer, dtype):
@@ -409,6 +454,16 @@ def run(args):
         return run_routed_experts(args, timer, dtype)
     elif args.kernel == "state_space":
         return run_state_space(args, timer, dtype)
+    elif args.kernel == "scaled_attention":
+        ms, nbytes, flops, extra = run_scaled_attention(args, timer)
+    elif args.kernel == "stream_norm":
+        s = args.streams
+        x, y = rand(args.tokens, s, args.hidden), rand(args.tokens, args.hidden).to(dtype)
+        mix, spread, gather = torch.eye(s, device="cuda") + 0.01 * rand(s, s), rand(s) * 0.1, rand(s)
+        gain, bias = rand(args.hidden), rand(args.hidden)
+        out = torch.empty((args.tokens, args.hidden), dtype=dtype, device="cuda")
+        ms = timer(lambda: ops.stream_norm(x, None, y, mix, spread, gather, gain, bias, 1e-6, out))
+        nbytes, flops = args.tokens * args.hidden * (8 * s + 2 * elem), 2.0 * args.tokens * args.hidden * s * (s + 2)
     elif args.kernel == "sum_layernorm":
         x, d1, d2 = rand(args.tokens, args.hidden), rand(args.tokens, args.hidden).to(dtype), \
             rand(args.tokens, args.hidden).to(dtype)
@@ -449,6 +504,10 @@ def main(argv=None) -> int:
     parser.add_argument("--k", type=int, default=3584)
     parser.add_argument("--nsplit", type=int, default=0, help="0 = the engine's choice")
     parser.add_argument("--state", type=int, default=128, help="state_space: state rows per head")
+    parser.add_argument("--streams", type=int, default=4, help="stream_norm: residual streams")
+    parser.add_argument("--chunk", type=int, default=0, help="scaled_attention: positions per chunk (0: none)")
+    parser.add_argument("--softcap", type=float, default=0.0, help="scaled_attention: cap on the scores (0: none)")
+    parser.add_argument("--gate", action="store_true", help="scaled_attention: a gate per column")
     parser.add_argument("--experts", type=int, default=64)
     parser.add_argument("--top", type=int, default=6)
     parser.add_argument("--groups", type=int, default=8)

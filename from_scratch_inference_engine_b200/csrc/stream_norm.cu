@@ -57,7 +57,7 @@ __device__ __forceinline__ void store4(bf16* p, const float (&v)[1]) { *p = __fl
 // STEP: columns per thread and trip (4: the width is a multiple of 4 and every row starts on 16
 // bytes, or 8 for bfloat16).
 template <typename T, int S, int STEP>
-__global__ void stream_norm_kernel(const StreamNormParams p) {
+__global__ void __launch_bounds__(512, S > 0 && S <= 4 ? 2 : 1) stream_norm_kernel(const StreamNormParams p) {
     extern __shared__ __align__(16) float sn_smem[];
     __shared__ float scratch[32];
     const int streams = S > 0 ? S : p.streams, width = p.width;
@@ -175,8 +175,9 @@ __global__ void stream_norm_kernel(const StreamNormParams p) {
 template <typename T, int S, int STEP>
 static int stream_norm_launch(const StreamNormParams& p, int num_rows, cudaStream_t stream) {
     const int columns = (p.width + STEP - 1) / STEP;
-    // few rows: as many threads as there is work for, so that a row is one trip to memory
-    const int threads = S == 0 ? 128 : (columns >= (num_rows <= 64 ? 512 : 1024) ? 512 : (columns >= 256 ? 256 : 128));
+    // few rows: as many threads as there is work for, so that a row is one trip to memory; many rows:
+    // smaller blocks, more of which fit beside one another
+    const int threads = S == 0 ? 128 : (num_rows <= 64 && columns >= 512 ? 512 : (columns >= 256 ? 256 : 128));
     const size_t floats = (size_t)((p.width + 3) & ~3) + (size_t)p.streams * p.streams + 2 * (size_t)p.streams +
                           (S == 0 ? (size_t)p.streams * threads : 0);
     const size_t smem = floats * sizeof(float);

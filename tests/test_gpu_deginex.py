@@ -283,7 +283,7 @@ class Attention:
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("dk,dv,kv_heads,chunk,softcap,gated", [
-    (24, 40, 2, 37, 6.0, True), (48, 48, 1, 200, 20.0, True), (48, 128, 2, 64, 3.0, True), (64, 64, 2, 100, 5.0, False),
+    (24, 40, 2, 37, 6.0, True), (80, 56, 1, 150, 17.0, True), (48, 128, 2, 64, 3.0, True), (64, 64, 2, 100, 5.0, False),
     (128, 128, 3, 128, 15.0, True), (64, 64, 6, 300, 0.0, True)])
 def test_capped_scores_chunks_and_gated_columns(dtype, dk, dv, kv_heads, chunk, softcap, gated):
     """Every form of the attention kernel that takes the sizes, whole and split over key ranges: a long

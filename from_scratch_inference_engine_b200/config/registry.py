@@ -15,6 +15,7 @@ from typing import Any, Dict, Mapping, Type
 
 from .deginex import DeginexConfig
 from .kufulix import KufulixConfig
+from .lanilorn import LanilornConfig
 from .metulix import MetulixConfig
 from .qwen2 import ConfigError, Qwen2Config
 from .tapalix import TapalixConfig
@@ -86,3 +87,4 @@ register_architecture("Zadepel", ZadepelConfig)
 register_architecture("Tapalix", TapalixConfig)
 register_architecture("Kufulix", KufulixConfig)
 register_architecture("Deginex", DeginexConfig)
+register_architecture("Lanilorn", LanilornConfig)

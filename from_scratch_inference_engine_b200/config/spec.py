@@ -51,6 +51,9 @@ class LayerSpec:
     feed_forward_out_norm: Optional[PartSpec] = None
     mixer_out_norm_name: str = "mixer_out_norm."
     feed_forward_out_norm_name: str = "feed_forward_out_norm."
+    # arrangements that multiply a sublayer's output column by column: the tensors' names below
+    # `prefix`, (the mixer's, the feed-forward's)
+    output_scale_names: Optional[Tuple[str, str]] = None
 
 
 @dataclass(frozen=True)

@@ -7,12 +7,15 @@ namespace fsie {
 // Merge the key splits of one (token, head); same arithmetic as attention_generic.cu.  The
 // weights e^(m_z - M) of splits z and z + 32 are computed once by lane z (nsplit <= 64) and
 // broadcast.  With `gate` (head h of token t at t * gate_ld + h * HD) the result is multiplied by its
-// sigmoid column by column before it is rounded.
+// sigmoid column by column before it is rounded, with `head_gate` (head h of token t at t * head_gate_ld + h)
+// by one sigmoid per head; with `sink` [heads] the denominator also holds e^(sink[h]).
 constexpr int MAX_KEY_SPLITS = 64;
 __global__ void attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                         bf16* __restrict__ out, int out_ld, int tokens, int heads,
                                         int nsplit, const int* __restrict__ token_list,
-                                        const bf16* __restrict__ gate, int gate_ld) {
+                                        const bf16* __restrict__ gate, int gate_ld,
+                                        const bf16* __restrict__ head_gate, int head_gate_ld,
+                                        const float* __restrict__ sink) {
     // the list of tokens was staged before the step: it is read while the attention kernel still runs
     const int tok = token_list ? token_list[blockIdx.x] : blockIdx.x, h = blockIdx.y;
     grid_dependency_wait();
@@ -42,8 +45,10 @@ __global__ void attn_combine_kernel(const float* __restrict__ part_o, const floa
     const float mmax = warp_max(fmaxf(mz, mz_hi));
     const float wz = mz == -INFINITY ? 0.f : __expf(mz - mmax);
     const float wz_hi = mz_hi == -INFINITY ? 0.f : __expf(mz_hi - mmax);
-    const float denom = warp_sum(lz * wz + lz_hi * wz_hi);
-    const float inv = denom > 0.f ? 1.0f / denom : 0.f;
+    float denom = warp_sum(lz * wz + lz_hi * wz_hi);
+    if (sink) denom += expf(sink[h] - mmax);
+    float inv = denom > 0.f ? 1.0f / denom : 0.f;
+    if (head_gate) inv *= 1.0f / (1.0f + expf(-__bfloat162float(head_gate[(size_t)tok * head_gate_ld + h])));
     // every lane of a warp takes every turn of this loop (the weights travel by shuffles); lanes
     // beyond the head's end - head sizes that are no multiple of 64 - load and store nothing
     for (int d0 = 0; d0 < HD; d0 += blockDim.x * 2) {

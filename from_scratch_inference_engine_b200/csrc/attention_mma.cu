@@ -450,7 +450,7 @@ int fsie_attn_mma(int row_class, const void* q, int q_ld, const void* k_pages, c
     if (nsplit > MAX_KEY_SPLITS) return ERR_BAD_ARGUMENT;
     return launch_dependent(attn_combine_kernel, cgrid, dim3(HD >= 128 ? 64 : 32), 0, stream,
                             (const float*)part_o, (const float*)part_ml, (bf16*)out, out_ld, tokens, heads, nsplit,
-                            combine_tokens, (const bf16*)nullptr, 0);
+                            combine_tokens, (const bf16*)nullptr, 0, (const bf16*)nullptr, 0, (const float*)nullptr);
 }
 
 }  // extern "C"

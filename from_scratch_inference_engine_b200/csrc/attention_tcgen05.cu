@@ -31,7 +31,10 @@
 // soon as they are read (CAP: through cap * tanh(s / cap) first), P is written as two bfloat16 halves -
 // the weight, and what rounding it lost - over both halves of the S columns, and O takes both; a
 // query may be confined to the keys of its own chunk of positions, and the result may be multiplied by
-// the sigmoid of a gate column by column before it is rounded.
+// the sigmoid of a gate, one per column or one per head, before it is rounded; the denominator may also hold
+// a sink per head, the scores have a factor per position of the query.  A key row may be two keys side by side
+// (`maps` = 2), each half as wide: a query head then is that narrow and reads one of them, its row zero
+// beside it; and the unmerged results of all key ranges may be left to the caller (`partial`).
 // Every wait on an mbarrier is bounded; when one runs out *error is set, all roles leave their
 // loops, tensor memory is freed and the kernel returns.
 #include "common.cuh"
@@ -80,6 +83,11 @@ struct TcExtra {
     int chunk;                         // > 0: a query sees only the keys of its own chunk of this many positions
     float softcap;                     // CAP: scores pass through softcap * tanh(s / softcap)
     const bf16* gate; int gate_ld;     // null, or head h of token t at t * gate_ld + h * HD
+    const bf16* head_gate; int head_gate_ld;   // null, or head h of token t at t * head_gate_ld + h
+    const float* sink;                 // null, or [heads]
+    const float* pos_scale; int pos_len;       // null, or a factor on the scores of the query at each position
+    int maps;                          // keys side by side in a key row (1 or 2)
+    int partial;                       // leave every key range's result, also of a single one, in part_o / part_ml
 };
 #define TC_MARK(slot) do { } while (0)
 
@@ -265,7 +273,13 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap pages_map, const AttnParams p
             if (e < CHUNKS && r < nrows) {
                 const int row = row0 + r;
                 const int tok = qstart + row / group, h = kvh * group + row % group;
-                held[j] = *reinterpret_cast<const uint4*>(q + (size_t)tok * p.q_ld + h * HD + c * 8);
+                if (WIDE && x.maps == 2) {
+                    const int at = c * 8 - (h & 1) * (HD / 2);              // zero beside the query's own key
+                    if (at >= 0 && at < HD / 2)
+                        held[j] = *reinterpret_cast<const uint4*>(q + (size_t)tok * p.q_ld + h * (HD / 2) + at);
+                } else {
+                    held[j] = *reinterpret_cast<const uint4*>(q + (size_t)tok * p.q_ld + h * HD + c * 8);
+                }
             }
         }
 #pragma unroll
@@ -396,7 +410,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap pages_map, const AttnParams p
         constexpr float LOG2E = 1.4426950408889634f;
         // WIDE: the scores are in base-2 units before anything is done with them
         const float sc = WIDE ? 1.f : p.scale * LOG2E;
-        const float natural = WIDE ? x.head_scale[kvh * group + (row0 + (valid ? st * BM + r : 0)) % group] : 0.f;
+        float natural = WIDE ? x.head_scale[kvh * group + (row0 + (valid ? st * BM + r : 0)) % group] : 0.f;
+        if (WIDE && x.pos_scale) natural *= x.pos_scale[min(max(pos, 0), x.pos_len - 1)];
         const float to_base2 = CAP ? 2.f * LOG2E * natural / x.softcap : LOG2E * natural;
         const float cap2 = CAP ? LOG2E * x.softcap : 0.f;
         float m_run = -INFINITY, l_run = 0.f;
@@ -521,7 +536,11 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap pages_map, const AttnParams p
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         const int row = row0 + (valid ? st * BM + r : 0);
         const int tok = qstart + row / group, h = kvh * group + row % group;
-        const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+        float denom = l_run;
+        if (WIDE && x.sink) denom += fast_exp2(x.sink[h] * LOG2E - m_run);
+        float inv = denom > 0.f ? 1.0f / denom : 0.f;
+        if (WIDE && x.head_gate) inv *= 1.0f / (1.0f + expf(-__bfloat162float(x.head_gate[(size_t)tok * x.head_gate_ld + h])));
+        const bool whole = p.nsplit == 1 && !(WIDE && x.partial);       // this range is all there is: the result itself
 #pragma unroll 1
         for (int c = 0; c < HD; c += 32) {
             float v[32];
@@ -531,7 +550,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap pages_map, const AttnParams p
                 for (int j = 0; j < 32; ++j) v[j] = 0.f;
             }
             if (!valid) continue;
-            if (p.nsplit == 1) {
+            if (whole) {
                 bf16* dst = (bf16*)p.out + (size_t)tok * p.out_ld + h * HD + c;
 #pragma unroll
                 for (int g8 = 0; g8 < 4; ++g8) {
@@ -556,7 +575,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap pages_map, const AttnParams p
                     *reinterpret_cast<float4*>(dst + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
             }
         }
-        if (valid && p.nsplit > 1) {
+        if (valid && !whole) {
             const size_t idx = ((size_t)split * p.tokens + tok) * p.heads + h;
             p.part_ml[idx * 2] = m_run == -INFINITY ? -INFINITY : m_run * (WIDE ? 0.6931471805599453f : p.scale);
             p.part_ml[idx * 2 + 1] = l_run;
@@ -1008,15 +1027,14 @@ static int attn_tc_launch(const void* pages_map, int entries, int entry, const v
                  const int* block_tables, int bt_stride, const int* tile_item, const int* tile_row0, int tiles,
                  const int* item_qstart, const int* item_qlen, const int* item_pos0, void* out, int out_ld,
                  float* part_o, float* part_ml, int tokens, int heads, int kv_heads, int head_dim, int window,
-                 int nsplit, float scale, const float* head_scale, int chunk, float softcap, const void* gate,
-                 int gate_ld, const int* combine_tokens, int num_combine, int* error, cudaStream_t stream) {
+                 int nsplit, float scale, const TcExtra& wide, const int* combine_tokens, int num_combine, int* error, cudaStream_t stream) {
     if (tiles <= 0 || tokens <= 0) return 0;
     if (head_dim != HD) return ERR_UNSUPPORTED;
     if (page_size != 8 && page_size != 16 && page_size != 32 && page_size != 64 && page_size != 128) return ERR_UNSUPPORTED;
     if (kv_heads <= 0 || heads % kv_heads != 0 || nsplit < 1 || nsplit > MAX_KEY_SPLITS || (q_ld % 8) != 0 ||
         (out_ld % 8) != 0 || entries <= 0 || entry < 0 || entry >= entries || !error)
         return ERR_BAD_ARGUMENT;
-    if (nsplit > 1 && (!part_o || !part_ml)) return ERR_BAD_ARGUMENT;
+    if ((nsplit > 1 || wide.partial) && (!part_o || !part_ml)) return ERR_BAD_ARGUMENT;
     CUtensorMap map;
     memcpy(&map, pages_map, sizeof(map));
     AttnParams p;
@@ -1028,9 +1046,10 @@ static int attn_tc_launch(const void* pages_map, int entries, int entry, const v
     p.out = out; p.out_ld = out_ld; p.part_o = part_o; p.part_ml = part_ml;
     p.tokens = tokens; p.heads = heads; p.kv_heads = kv_heads; p.head_dim = head_dim;
     p.window = window; p.nsplit = nsplit; p.scale = scale;
-    TcExtra x;
+    TcExtra x = wide;
     x.entries = entries; x.entry = entry; x.error = error;
-    x.head_scale = head_scale; x.chunk = chunk; x.softcap = softcap; x.gate = (const bf16*)gate; x.gate_ld = gate_ld;
+    const float* head_scale = x.head_scale;
+    const float softcap = x.softcap;
     auto* kernel = !head_scale ? attn_tc_kernel<false, false>
                                : (softcap > 0.f ? attn_tc_kernel<true, true> : attn_tc_kernel<true, false>);
     const int form = !head_scale ? 0 : (softcap > 0.f ? 2 : 1);
@@ -1042,11 +1061,12 @@ static int attn_tc_launch(const void* pages_map, int entries, int entry, const v
     }
     kernel<<<dim3(tiles * kv_heads, 1, nsplit), THREADS, SMEM_BYTES, stream>>>(map, p, x);
     int rc = (int)cudaGetLastError();
-    if (rc != 0 || nsplit == 1) return rc;
+    if (rc != 0 || nsplit == 1 || x.partial) return rc;
     const int count = combine_tokens ? num_combine : tokens;
     if (count <= 0) return 0;
     attn_combine_kernel<<<dim3(count, heads), HD >= 128 ? 64 : 32, 0, stream>>>(
-        part_o, part_ml, (bf16*)out, out_ld, tokens, heads, nsplit, combine_tokens, (const bf16*)gate, gate_ld);
+        part_o, part_ml, (bf16*)out, out_ld, tokens, heads, nsplit, combine_tokens, x.gate, x.gate_ld, x.head_gate,
+        x.head_gate_ld, x.sink);
     return (int)cudaGetLastError();
 }
 
@@ -1058,25 +1078,34 @@ int fsie_attn_tc(const void* pages_map, int entries, int entry, const void* q, i
                  cudaStream_t stream) {
     return attn_tc_launch(pages_map, entries, entry, q, q_ld, page_size, block_tables, bt_stride, tile_item, tile_row0,
                           tiles, item_qstart, item_qlen, item_pos0, out, out_ld, part_o, part_ml, tokens, heads,
-                          kv_heads, head_dim, window, nsplit, scale, nullptr, 0, 0.f, nullptr, 0, combine_tokens,
-                          num_combine, error, stream);
+                          kv_heads, head_dim, window, nsplit, scale, TcExtra{}, combine_tokens, num_combine, error,
+                          stream);
 }
 
 // The WIDE form: weights as two bfloat16 halves, a scale per head (head_scale [heads], float), chunk > 0:
 // keys of the query's own chunk only, softcap > 0: capped scores, gate (null, or heads x head_dim columns
-// per token, rows gate_ld apart, on 16-byte borders): the result times its sigmoid.
+// per token, rows gate_ld apart, on 16-byte borders): the result times its sigmoid; head_gate (null, or one
+// number per head and token, rows head_gate_ld apart), sink (null or [heads]), pos_scale (null, or [pos_len]
+// factors by the query's position), maps (1 or 2) and partial: see the head of this file.  `heads` counts
+// every map's query heads.
 int fsie_attn_tc_scaled(const void* pages_map, int entries, int entry, const void* q, int q_ld, int page_size,
                         const int* block_tables, int bt_stride, const int* tile_item, const int* tile_row0, int tiles,
                         const int* item_qstart, const int* item_qlen, const int* item_pos0, void* out, int out_ld,
                         float* part_o, float* part_ml, int tokens, int heads, int kv_heads, int head_dim, int window,
                         int nsplit, const float* head_scale, int chunk, float softcap, const void* gate, int gate_ld,
-                        const int* combine_tokens, int num_combine, int* error, cudaStream_t stream) {
-    if (!head_scale || chunk < 0 || !(softcap >= 0.f) || (gate && (gate_ld % 8 || ((size_t)gate & 15))))
+                        const void* head_gate, int head_gate_ld, const float* sink, const float* pos_scale,
+                        int pos_len, int maps, int partial, const int* combine_tokens, int num_combine, int* error,
+                        cudaStream_t stream) {
+    if (!head_scale || chunk < 0 || !(softcap >= 0.f) || (gate && (gate_ld % 8 || ((size_t)gate & 15))) ||
+        maps < 1 || maps > 2 || (kv_heads > 0 && heads % (kv_heads * maps) != 0) || (pos_scale && pos_len <= 0))
         return ERR_BAD_ARGUMENT;
+    TcExtra x = {};
+    x.head_scale = head_scale; x.chunk = chunk; x.softcap = softcap; x.gate = (const bf16*)gate; x.gate_ld = gate_ld;
+    x.head_gate = (const bf16*)head_gate; x.head_gate_ld = head_gate_ld; x.sink = sink; x.pos_scale = pos_scale;
+    x.pos_len = pos_len; x.maps = maps; x.partial = partial;
     return attn_tc_launch(pages_map, entries, entry, q, q_ld, page_size, block_tables, bt_stride, tile_item, tile_row0,
                           tiles, item_qstart, item_qlen, item_pos0, out, out_ld, part_o, part_ml, tokens, heads,
-                          kv_heads, head_dim, window, nsplit, 0.f, head_scale, chunk, softcap, gate, gate_ld,
-                          combine_tokens, num_combine, error, stream);
+                          kv_heads, head_dim, window, nsplit, 0.f, x, combine_tokens, num_combine, error, stream);
 }
 
 // Tiles of up to 16 query rows (decoded tokens, two-token portions): attn_tc_decode_kernel.
@@ -1107,7 +1136,7 @@ int fsie_attn_tc_decode(const void* pages_map, int entries, int entry, const voi
     p.out = out; p.out_ld = out_ld; p.part_o = part_o; p.part_ml = part_ml;
     p.tokens = tokens; p.heads = heads; p.kv_heads = kv_heads; p.head_dim = head_dim;
     p.window = window; p.nsplit = nsplit; p.scale = scale;
-    TcExtra x;
+    TcExtra x = {};
     x.entries = entries; x.entry = entry; x.error = error;
     static bool configured = false;
     if (!configured) {
@@ -1122,7 +1151,7 @@ int fsie_attn_tc_decode(const void* pages_map, int entries, int entry, const voi
     if (count <= 0) return 0;
     return launch_dependent(attn_combine_kernel, dim3(count, heads), dim3(HD >= 128 ? 64 : 32), 0, stream,
                             (const float*)part_o, (const float*)part_ml, (bf16*)out, out_ld, tokens, heads, nsplit,
-                            combine_tokens, (const bf16*)nullptr, 0);
+                            combine_tokens, (const bf16*)nullptr, 0, (const bf16*)nullptr, 0, (const float*)nullptr);
 }
 #else
 int fsie_attn_tc_decode_rows() { return 0; }

@@ -39,7 +39,7 @@ struct GemmParams {
     const bf16* bias;               // [N] or null
     int T, N, K;                    // N = output features (SwiGLU: intermediate size)
     int up_row0;                    // SwiGLU: row of w where the up rows start
-    int gate;                       // gated epilogue: 1 = SiLU on the gate, 2 = GELU (tanh form)
+    int gate;                       // gated epilogue: 1 = SiLU on the gate, 2 = GELU (tanh form); plain epilogue: 3 = the square of relu on the result
     int kblocks_per_split;
     int out_f32;
     int* error;
@@ -254,6 +254,10 @@ gemm_decode_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
                                : g / (1.0f + expf(-g))) * u;
         } else {
             out = acc + (p.bias ? __bfloat162float(p.bias[n]) : 0.f);
+            if (p.gate == 3) {                // no gate, the square of relu: on the value as bfloat16 would store it
+                const float r = fmaxf(__bfloat162float(__float2bfloat16_rn(out)), 0.f);
+                out = r * r;
+            }
         }
         if (p.out_f32) reinterpret_cast<float*>(p.y)[(size_t)t * p.ldy + n] = out;
         else reinterpret_cast<bf16*>(p.y)[(size_t)t * p.ldy + n] = __float2bfloat16_rn(out);
@@ -327,13 +331,14 @@ int fsie_gemm_decode_weight_map(void* map_out, const void* w, long long rows, lo
 }
 
 // y[T, N] = x[T, K] * w^T (+ bias), or for swiglu != 0 y[T, N] = act(x w_gate^T) * (x w_up^T) with
-// w = [gate rows (N); up rows (N)], act = SiLU (swiglu = 1) or the tanh form of GELU (2).  T <= 64.  `splits` (1, 2, 4 or 8) cuts K over a cluster.
+// w = [gate rows (N); up rows (N)], act = SiLU (swiglu = 1) or the tanh form of GELU (2); swiglu = 3: no gate, y = relu(x w^T)^2.  T <= 64.  `splits` (1, 2, 4 or 8) cuts K over a cluster.
 int fsie_gemm_decode(const void* weight_map, const void* x, int ldx, void* y, int ldy, const void* bias,
                      int T, int N, int K, int swiglu, int out_f32, int splits, int* error, cudaStream_t stream) {
     if (T <= 0 || N <= 0) return 0;
     if (T > 64 || K <= 0 || K % 8 != 0 || ldx % 8 != 0 || (splits != 1 && splits != 2 && splits != 4 && splits != 8) ||
-        swiglu < 0 || swiglu > 2)
+        swiglu < 0 || swiglu > 3)
         return ERR_BAD_ARGUMENT;
+    const bool gated = swiglu == 1 || swiglu == 2;
     const int TN = T <= 16 ? 16 : (T <= 32 ? 32 : 64);
     CUtensorMap map_w, map_x;
     memcpy(&map_w, weight_map, sizeof(map_w));
@@ -344,9 +349,9 @@ int fsie_gemm_decode(const void* weight_map, const void* x, int ldx, void* y, in
     p.up_row0 = N; p.out_f32 = out_f32; p.error = error; p.gate = swiglu;
     const int total_kblocks = (K + BK - 1) / BK;
     p.kblocks_per_split = (total_kblocks + splits - 1) / splits;
-    const int tiles = swiglu ? (N + BM / 2 - 1) / (BM / 2) : (N + BM - 1) / BM;
+    const int tiles = gated ? (N + BM / 2 - 1) / (BM / 2) : (N + BM - 1) / BM;
 #define FSIE_GEMM(TNV)                                                                             \
-    (swiglu ? launch<TNV, EPI_SWIGLU>(map_w, map_x, p, tiles, splits, stream)                      \
+    (gated ? launch<TNV, EPI_SWIGLU>(map_w, map_x, p, tiles, splits, stream)                      \
             : launch<TNV, EPI_PLAIN>(map_w, map_x, p, tiles, splits, stream))
     if (TN == 16) rc = FSIE_GEMM(16);
     else if (TN == 32) rc = FSIE_GEMM(32);

@@ -27,7 +27,7 @@ constexpr int SK_AHEAD = 4;          // chunks whose weights a warp has asked fo
 struct SkinnyParams {
     const bf16* w; const bf16* x; long long ldx;
     void* y; long long ldy; const bf16* bias;
-    int T, N, K, out_f32;
+    int T, N, K, out_f32, relu2;
 };
 
 // The q, k, v product of an attention layer with what follows it on the way to the cache: w
@@ -219,6 +219,10 @@ gemm_skinny_kernel(const SkinnyParams p, const SkinnyRope rope) {
 #pragma unroll
         for (int w = 0; w < SK_WARPS; ++w) sum += red[((size_t)w * SK_ROWS + r) * TP + token];
         if (p.bias) sum += __bfloat162float(p.bias[n]);
+        if (p.relu2) {                        // the square of relu, on the value as bfloat16 would store it
+            const float r = fmaxf(__bfloat162float(__float2bfloat16_rn(sum)), 0.f);
+            sum = r * r;
+        }
         if (p.out_f32) reinterpret_cast<float*>(p.y)[(size_t)token * p.ldy + n] = sum;
         else reinterpret_cast<bf16*>(p.y)[(size_t)token * p.ldy + n] = __float2bfloat16_rn(sum);
     }
@@ -244,15 +248,16 @@ using namespace fsie;
 extern "C" {
 
 // y[T, N] = x[T, K] * w^T (+ bias); T <= 16, K a multiple of 32, rows of x and w on 16-byte boundaries.
+// relu2 != 0: the square of relu of the result, taken as bfloat16 would store it.
 int fsie_gemm_skinny(const void* w, const void* x, long long ldx, void* y, long long ldy, const void* bias,
-                     int T, int N, int K, int out_f32, cudaStream_t stream) {
+                     int T, int N, int K, int out_f32, int relu2, cudaStream_t stream) {
     if (T <= 0 || N <= 0) return 0;
     if (T > 16 || K <= 0 || K % SK_CHUNK != 0 || ldx % 8 != 0 || (reinterpret_cast<uintptr_t>(w) & 15) ||
         (reinterpret_cast<uintptr_t>(x) & 15))
         return ERR_BAD_ARGUMENT;
     SkinnyParams p;
     p.w = (const bf16*)w; p.x = (const bf16*)x; p.ldx = ldx; p.y = y; p.ldy = ldy; p.bias = (const bf16*)bias;
-    p.T = T; p.N = N; p.K = K; p.out_f32 = out_f32;
+    p.T = T; p.N = N; p.K = K; p.out_f32 = out_f32; p.relu2 = relu2;
     SkinnyRope none = {};
     return T <= 8 ? launch_skinny<1, false>(p, none, stream) : launch_skinny<2, false>(p, none, stream);
 }
@@ -272,7 +277,7 @@ int fsie_gemm_skinny_qkv_rope(const void* w, const void* x, long long ldx, void*
         return ERR_BAD_ARGUMENT;
     SkinnyParams p;
     p.w = (const bf16*)w; p.x = (const bf16*)x; p.ldx = ldx; p.y = q_out; p.ldy = ldq; p.bias = (const bf16*)bias;
-    p.T = T; p.N = (heads + 2 * kv_heads) * head_dim; p.K = K; p.out_f32 = 0;
+    p.T = T; p.N = (heads + 2 * kv_heads) * head_dim; p.K = K; p.out_f32 = 0; p.relu2 = 0;
     SkinnyRope rope;
     rope.positions = positions; rope.cos_sin = cos_sin; rope.table_len = table_len;
     rope.slot_of = k_pages ? slot_of : nullptr; rope.k_pages = (bf16*)k_pages; rope.v_pages = (bf16*)v_pages;

@@ -168,6 +168,25 @@ __global__ void gated_act_vec_kernel(const T* __restrict__ gu, T* __restrict__ a
     store8(act + t * inter + i, o);
 }
 
+// x[i] <- relu(x[i])^2 in place, for products whose kernel has no such epilogue.  VEC: eight elements per thread.
+template <typename T, bool VEC>
+__global__ void relu_squared_kernel(T* __restrict__ x, long long count) {
+    grid_dependency_wait();
+    grid_dependents_go();
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= count) return;
+    if (VEC) {
+        float v[8];
+        load8(x + i * 8, v);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) { const float r = fmaxf(v[e], 0.f); v[e] = r * r; }
+        store8(x + i * 8, v);
+    } else {
+        const float r = fmaxf(to_float(x[i]), 0.f);
+        x[i] = from_float<T>(r * r);
+    }
+}
+
 template <typename T>
 static int norm_add_norm_launch(float* x, const void* delta, const float* gain_d, const float* gain,
                                 void* y, const int* rows, int num_rows, int hidden, float eps_d,
@@ -302,6 +321,19 @@ int fsie_gated_act(const void* gu, void* act, long long tokens, int inter, int k
                                 (const float*)gu, (float*)act, inter, total, kind);
     return launch_dependent(gated_act_kernel<bf16>, dim3(blocks), dim3(threads), 0, stream,
                             (const bf16*)gu, (bf16*)act, inter, total, kind);
+}
+
+// x [count] of storage type `dtype`, squared where positive and zero elsewhere, in place.
+int fsie_relu_squared(void* x, long long count, int dtype, cudaStream_t stream) {
+    if (count <= 0) return 0;
+    const bool vec = count % 8 == 0 && (((size_t)x) & 31) == 0;
+    const long long work = vec ? count / 8 : count;
+    const long long blocks = (work + 255) / 256;
+    if (blocks > 0x7fffffffLL) return ERR_UNSUPPORTED;
+#define FSIE_RELU2(T, V) launch_dependent(relu_squared_kernel<T, V>, dim3((unsigned)blocks), dim3(256), 0, stream, (T*)x, work)
+    if (dtype == DTYPE_F32) return vec ? FSIE_RELU2(float, true) : FSIE_RELU2(float, false);
+    return vec ? FSIE_RELU2(bf16, true) : FSIE_RELU2(bf16, false);
+#undef FSIE_RELU2
 }
 
 // x float32 [*, hidden]; d1, d2 and y of storage type `dtype` (any may be null); gain float32 [hidden].

@@ -8,7 +8,15 @@
 //                                                       and (chunk == 0 or i / chunk == j / chunk)
 //   softcap > 0:  s_h(i, j) <- softcap * tanh(s_h(i, j) / softcap)
 //   o_h,i     = sum_j softmax_j(s_h(i, .)) v_g(h),j      g(h) = h / (heads / kv_heads)
-//   with gates:   o_h,i <- o_h,i * sigmoid(gate_h,i)     column by column, before the result is rounded
+//   with gates:   o_h,i <- o_h,i * sigmoid(gate_h,i)     column by column, or one number per head, before the
+//                                                       result is rounded
+//   with sinks:   the softmax's denominator also holds e^(sink_h), which has no key and no value
+//   pos_scale:    s_h(i, j) is multiplied by pos_scale[i], one number per position of a query
+//   maps > 1:     a key row is `maps` keys side by side, each key_dim / maps wide, over ONE value row; query
+//                 head h (of `maps` times as many) is that narrow and reads key h % maps of its key/value
+//                 head.  Its row enters the products as wide as the key row, zero beside its own key.
+//   partial:      the maximum, the sum and the unnormalised output of every key range are left to the
+//                 caller, also of a single range (fsie_difference_merge reads them)
 //
 // Work is cut as in attention_generic.cu: a tile is up to ROWS query rows of one request and one
 // key/value head, a row being (token, head of the group): row = token * group + head_in_group; a
@@ -42,6 +50,11 @@ struct ScaledAttnParams {
     int chunk;                                // > 0: a query sees only the keys of its own chunk of this many positions
     float softcap;                            // > 0: scores pass through softcap * tanh(s / softcap)
     const void* gate; int gate_ld;            // null, or head h of token t at t * gate_ld + h * value_dim
+    const void* head_gate; int head_gate_ld;  // null, or head h of token t at t * head_gate_ld + h
+    const float* sink;                        // null, or [heads]
+    const float* pos_scale; int pos_len;      // null, or a factor on the scores of the query at each position
+    int maps, q_dim;                          // keys side by side in a key row; columns of a query (key_dim / maps)
+    int partial;
     int page_shift;                           // log2(page_size), or -1 where it is no power of two
     int* error;
 };
@@ -60,6 +73,29 @@ __device__ __forceinline__ float sa_cap_fast(float s, float cap, float twice_inv
 }
 
 __device__ __forceinline__ float sa_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+// What a row's scores are multiplied by: its head's scale, and its position's where there is one.
+__device__ __forceinline__ float sa_row_scale(const ScaledAttnParams& p, int head, int pos) {
+    float sc = p.head_scale[head];
+    if (p.pos_scale) sc *= p.pos_scale[min(max(pos, 0), p.pos_len - 1)];
+    return sc;
+}
+
+// Where column c of the key row's width lies in head h's query, or -1: another map's column, zero.
+__device__ __forceinline__ int sa_query_column(const ScaledAttnParams& p, int head, int c) {
+    const int at = c - (p.maps > 1 ? (head % p.maps) * p.q_dim : 0);
+    return at >= 0 && at < p.q_dim ? at : -1;
+}
+
+// One over a row's softmax denominator - `total` and the head's sink, relative to e^m - times its head's gate.
+template <typename T>
+__device__ __forceinline__ float sa_row_factor(float total, float m, const float* sink, const void* head_gate,
+                                               int head_gate_ld, int tok, int head) {
+    if (sink) total += expf(sink[head] - m);
+    float f = total > 0.f ? 1.0f / total : 0.f;
+    if (head_gate) f *= sa_sigmoid(to_float(((const T*)head_gate)[(size_t)tok * head_gate_ld + head]));
+    return f;
+}
 
 template <typename T, int DPL, bool SHARED_V>
 __global__ void __launch_bounds__(SA_WARPS * 32) scaled_attention_kernel(const ScaledAttnParams p) {
@@ -92,9 +128,11 @@ __global__ void __launch_bounds__(SA_WARPS * 32) scaled_attention_kernel(const S
     for (int r = warp; r < SA_ROWS; r += SA_WARPS) {
         const int row = row0 + r;
         const int tok = qstart + row / group, h = kvh * group + row % group;
-        const float sc = r < nrows ? p.head_scale[h] : 0.f;
-        for (int d = lane; d < dk4; d += 32)
-            qs[r * dk4 + d] = (r < nrows && d < dk) ? to_float(q[(size_t)tok * p.q_ld + (size_t)h * dk + d]) * sc : 0.f;
+        const float sc = r < nrows ? sa_row_scale(p, h, pos0 + row / group) : 0.f;
+        for (int d = lane; d < dk4; d += 32) {
+            const int at = sa_query_column(p, h, d);
+            qs[r * dk4 + d] = (r < nrows && at >= 0) ? to_float(q[(size_t)tok * p.q_ld + (size_t)h * p.q_dim + at]) * sc : 0.f;
+        }
     }
 
     const int pos_first = pos0 + row0 / group;
@@ -213,9 +251,9 @@ __global__ void __launch_bounds__(SA_WARPS * 32) scaled_attention_kernel(const S
         if (r >= nrows) continue;
         const int row = row0 + r;
         const int tok = qstart + row / group, h = kvh * group + row % group;
-        if (p.nsplit == 1) {
+        if (p.nsplit == 1 && !p.partial) {
             T* o = (T*)p.out + (size_t)tok * p.out_ld + (size_t)h * dv;
-            const float inv = l[i] > 0.f ? 1.0f / l[i] : 0.f;
+            const float inv = sa_row_factor<T>(l[i], m[i], p.sink, p.head_gate, p.head_gate_ld, tok, h);
 #pragma unroll
             for (int c = 0; c < DPL; ++c) {
                 const int d = lane + 32 * c;
@@ -377,10 +415,12 @@ __global__ void __launch_bounds__(SA_WARPS * 32) scaled_attention_mma_kernel(con
     // the tile's query rows as they are (the head's scale meets the scores), zero beyond the tile
     for (int r = warp; r < SA_ROWS; r += SA_WARPS) {
         const int row = row0 + r;
-        const bf16* src = q + (size_t)(qstart + row / group) * p.q_ld + (size_t)(kvh * group + row % group) * dk;
+        const int h = kvh * group + row % group;
+        const bf16* src = q + (size_t)(qstart + row / group) * p.q_ld + (size_t)h * p.q_dim;
         for (int c = lane; c < dk / 8; c += 32) {
             uint4 v = make_uint4(0u, 0u, 0u, 0u);
-            if (r < nrows) v = *reinterpret_cast<const uint4*>(src + c * 8);
+            const int at = sa_query_column(p, h, c * 8);
+            if (r < nrows && at >= 0) v = *reinterpret_cast<const uint4*>(src + at);
             *reinterpret_cast<uint4*>(Qs + r * L.ldk + c * 8) = v;
         }
     }
@@ -393,7 +433,7 @@ __global__ void __launch_bounds__(SA_WARPS * 32) scaled_attention_mma_kernel(con
         const int r = mi * 16 + g + 8 * i;
         pos[i] = r < nrows ? pos0 + (row0 + r) / group : -1;
         first_key[i] = sa_first_key(p, pos[i]);
-        sc[i] = r < nrows ? p.head_scale[kvh * group + (row0 + r) % group] : 0.f;
+        sc[i] = r < nrows ? sa_row_scale(p, kvh * group + (row0 + r) % group, pos[i]) : 0.f;
         m[i] = -INFINITY; l[i] = 0.f;
     }
     const float cap_inv = p.softcap > 0.f ? 2.0f / p.softcap : 0.f;
@@ -523,8 +563,8 @@ __global__ void __launch_bounds__(SA_WARPS * 32) scaled_attention_mma_kernel(con
         const float total = (q4.x + q4.y) + (q4.z + q4.w);
         const int row = row0 + r;
         const int tok = qstart + row / group, h = kvh * group + row % group;
-        if (p.nsplit == 1) {
-            const float inv = total > 0.f ? 1.0f / total : 0.f;
+        if (p.nsplit == 1 && !p.partial) {
+            const float inv = sa_row_factor<bf16>(total, m[i], p.sink, p.head_gate, p.head_gate_ld, tok, h);
             bf16* o = (bf16*)p.out + (size_t)tok * p.out_ld + (size_t)h * dv + vi * dvq + 2 * t;
             const bf16* gr = p.gate ? (const bf16*)p.gate + (size_t)tok * p.gate_ld + (size_t)h * dv + vi * dvq + 2 * t : nullptr;
 #pragma unroll
@@ -655,10 +695,12 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
 
     for (int r = warp; r < ROWS; r += TR_WARPS) {
         const int row = row0 + r;
-        const bf16* src = q + (size_t)(qstart + row / group) * p.q_ld + (size_t)(kvh * group + row % group) * dk;
+        const int h = kvh * group + row % group;
+        const bf16* src = q + (size_t)(qstart + row / group) * p.q_ld + (size_t)h * p.q_dim;
         for (int c = lane; c < dk / 8; c += 32) {
             uint4 v = make_uint4(0u, 0u, 0u, 0u);
-            if (r < nrows) v = *reinterpret_cast<const uint4*>(src + c * 8);
+            const int at = sa_query_column(p, h, c * 8);
+            if (r < nrows && at >= 0) v = *reinterpret_cast<const uint4*>(src + at);
             *reinterpret_cast<uint4*>(Qs + r * L.ldk + c * 8) = v;
         }
     }
@@ -670,7 +712,7 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
         const int r = wrow + g + 8 * i;
         pos[i] = r < nrows ? pos0 + (row0 + r) / group : -1;
         first_key[i] = sa_first_key(p, pos[i]);
-        sc[i] = r < nrows ? p.head_scale[kvh * group + (row0 + r) % group] : 0.f;
+        sc[i] = r < nrows ? sa_row_scale(p, kvh * group + (row0 + r) % group, pos[i]) : 0.f;
         m[i] = -INFINITY; l[i] = 0.f;
     }
     // the latest position among this warp's rows: tiles of keys beyond it are none of its business
@@ -818,8 +860,8 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
             }
             const int row = row0 + r;
             const int tok = qstart + row / group, h = kvh * group + row % group;
-            if (p.nsplit == 1) {
-                const float inv = total > 0.f ? 1.0f / total : 0.f;
+            if (p.nsplit == 1 && !p.partial) {
+                const float inv = sa_row_factor<bf16>(total, mmax, p.sink, p.head_gate, p.head_gate_ld, tok, h);
                 const bf16* gate = p.gate ? (const bf16*)p.gate + (size_t)tok * p.gate_ld + (size_t)h * dv + d : nullptr;
                 *reinterpret_cast<__nv_bfloat162*>((bf16*)p.out + (size_t)tok * p.out_ld + (size_t)h * dv + d) =
                     sa_gated_pair(a * inv, b * inv, gate);
@@ -839,8 +881,8 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
         if (r >= nrows) continue;
         const int row = row0 + r;
         const int tok = qstart + row / group, h = kvh * group + row % group;
-        if (p.nsplit == 1) {
-            const float inv = l[i] > 0.f ? 1.0f / l[i] : 0.f;
+        if (p.nsplit == 1 && !p.partial) {
+            const float inv = sa_row_factor<bf16>(l[i], m[i], p.sink, p.head_gate, p.head_gate_ld, tok, h);
             bf16* o = (bf16*)p.out + (size_t)tok * p.out_ld + (size_t)h * dv + 2 * t;
             const bf16* gr = p.gate ? (const bf16*)p.gate + (size_t)tok * p.gate_ld + (size_t)h * dv + 2 * t : nullptr;
 #pragma unroll
@@ -858,6 +900,18 @@ __global__ void __launch_bounds__(TR_WARPS * 32) scaled_attention_rows_kernel(co
     }
 }
 
+__device__ __forceinline__ void sa_load(const float* p, float (&v)[4]) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+__device__ __forceinline__ void sa_load(const float* p, float (&v)[1]) { v[0] = *p; }
+__device__ __forceinline__ void sa_store(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void sa_store(bf16* p, const float (&v)[4]) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+template <typename T> __device__ __forceinline__ void sa_store(T* p, const float (&v)[1]) { *p = from_float<T>(v[0]); }
+
 // o = sum_z acc_z e^(m_z - M) / sum_z l_z e^(m_z - M) over the key ranges z of one (token, head).  The
 // weights of 32 ranges at a time are worked out by the lanes of every warp and handed round by shuffles;
 // a range's values are asked for eight ranges at a time.
@@ -865,7 +919,8 @@ template <typename T>
 __global__ void sa_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                   T* __restrict__ out, int out_ld, int tokens, int heads, int dv,
                                   int nsplit, const T* __restrict__ gate, int gate_ld,
-                                  const int* __restrict__ token_list) {
+                                  const T* __restrict__ head_gate, int head_gate_ld,
+                                  const float* __restrict__ sink, const int* __restrict__ token_list) {
     // the list of tokens was staged before the step: it is read while the attention kernel still runs
     const int tok = token_list ? token_list[blockIdx.x] : blockIdx.x, h = blockIdx.y;
     const int lane = threadIdx.x & 31;
@@ -905,9 +960,96 @@ __global__ void sa_combine_kernel(const float* __restrict__ part_o, const float*
             }
         }
         if (!mine) continue;
-        o *= denom > 0.f ? 1.0f / denom : 0.f;
+        o *= sa_row_factor<T>(denom, mmax, sink, head_gate, head_gate_ld, tok, h);
         if (gate) o *= sa_sigmoid(to_float(gate[(size_t)tok * gate_ld + (size_t)h * dv + d]));
         out[(size_t)tok * out_ld + (size_t)h * dv + d] = from_float<T>(o);
+    }
+}
+
+// The difference of two softmax maps over the same values, from what the attention left of every key range
+// (`partial`; map m of head h is query head 2 h + m there):
+//   a_m = sum_z acc_m,z e^(m_m,z - M_m) / sum_z l_m,z e^(m_m,z - M_m)         over the key ranges z
+//   o   = a_1 - lambda a_2;   out = T( o / sqrt(mean(o^2) + eps) * factor * sigmoid(gate_h) )
+// A warp owns one (token, head); VEC columns side by side per lane and trip, NC trips.
+template <typename T, int VEC, int NC>
+__global__ void __launch_bounds__(128) difference_merge_kernel(
+        const float* __restrict__ part_o, const float* __restrict__ part_ml, T* __restrict__ out, int out_ld,
+        int tokens, int heads, int dv, int nsplit, float lambda, float eps, float factor, const T* __restrict__ gate,
+        int gate_ld, const int* __restrict__ token_list, int count) {
+    const int lane = threadIdx.x & 31;
+    const long long pair = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (pair >= (long long)count * heads) return;
+    const int listed = (int)(pair / heads), h = (int)(pair - (long long)listed * heads);
+    const int tok = token_list ? token_list[listed] : listed;       // (staged before the step)
+    grid_dependency_wait();
+    grid_dependents_go();
+    const size_t stride = (size_t)tokens * heads * 2, slot = ((size_t)tok * heads + h) * 2;
+    float o[NC][VEC];
+#pragma unroll
+    for (int map = 0; map < 2; ++map) {
+        float acc[NC][VEC];
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+#pragma unroll
+            for (int x = 0; x < VEC; ++x) acc[c][x] = 0.f;
+        float mmax = -INFINITY, denom = 0.f;
+        for (int z0 = 0; z0 < nsplit; z0 += 32) {
+            float mz = -INFINITY, lz = 0.f;
+            if (z0 + lane < nsplit) {
+                const float2 ml = *reinterpret_cast<const float2*>(part_ml + ((size_t)(z0 + lane) * stride + slot + map) * 2);
+                mz = ml.x;
+                lz = ml.y;
+            }
+            const float m_new = fmaxf(mmax, warp_max(mz));
+            const float corr = mmax == -INFINITY ? 0.f : expf(mmax - m_new);
+            const float w = mz == -INFINITY ? 0.f : expf(mz - m_new);
+            mmax = m_new;
+            denom = denom * corr + warp_sum(lz * w);
+#pragma unroll
+            for (int c = 0; c < NC; ++c)
+#pragma unroll
+                for (int x = 0; x < VEC; ++x) acc[c][x] *= corr;
+            const int n = min(32, nsplit - z0);
+#pragma unroll 4
+            for (int j = 0; j < n; ++j) {
+                const float wj = __shfl_sync(0xffffffffu, w, j);
+                const float* row = part_o + ((size_t)(z0 + j) * stride + slot + map) * dv;
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    const int d = (lane + 32 * c) * VEC;
+                    if (d >= dv) continue;
+                    float v[VEC];
+                    sa_load(row + d, v);
+#pragma unroll
+                    for (int x = 0; x < VEC; ++x)
+                        if (wj != 0.f) acc[c][x] += v[x] * wj;      // a range without keys may hold anything
+                }
+            }
+        }
+        const float inv = denom > 0.f ? 1.0f / denom : 0.f;
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+#pragma unroll
+            for (int x = 0; x < VEC; ++x) {
+                if (map == 0) o[c][x] = acc[c][x] * inv;
+                else o[c][x] -= lambda * (acc[c][x] * inv);
+            }
+    }
+    float sq = 0.f;
+#pragma unroll
+    for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int x = 0; x < VEC; ++x) sq += o[c][x] * o[c][x];      // columns beyond dv are zero
+    float f = factor / sqrtf(warp_sum(sq) / (float)dv + eps);
+    if (gate) f *= sa_sigmoid(to_float(gate[(size_t)tok * gate_ld + h]));
+    T* dst = out + (size_t)tok * out_ld + (size_t)h * dv;
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+        const int d = (lane + 32 * c) * VEC;
+        if (d >= dv) continue;
+#pragma unroll
+        for (int x = 0; x < VEC; ++x) o[c][x] *= f;
+        sa_store(dst + d, o[c]);
     }
 }
 
@@ -977,9 +1119,12 @@ __global__ void rotate_mix_write_kernel(T* __restrict__ proj, int ld, const int*
 // a warp per head of q and k in turn.
 //   q, k   with gains (q_gain, k_gain [dim], shared by the heads): every head divided by its root
 //          mean square (eps inside the root) times the gain, in 32-bit, BEFORE the rotation; with
-//          `unit` a side without a gain is divided by its root mean square alone;
+//          `unit` a side without a gain is divided by its root mean square alone; with `whole` the root
+//          mean square is over all heads of q (of k) at once and a gain holds a number per column of
+//          all of them;
 //          then pairs (i, i + rotary_dim / 2) turn by the token's angles; q in place, k into its page
-//   v      into its page as it is
+//   v      into its page as it is; with `v_from_k` the projection holds no v, and the values are the
+//          keys as they were projected (vdim = dim)
 // VEC: head sizes are multiples of 8 and every row and page starts on 16 bytes: eight
 // columns per lane and trip.
 template <typename T, bool VEC>
@@ -989,8 +1134,9 @@ __global__ void norm_rotate_write_kernel(T* __restrict__ proj, int ld, const int
                                          T* __restrict__ v_pages, long long page_stride, int page_size,
                                          int heads, int kv_heads, int dim, int vdim, int rotary_dim,
                                          const float* __restrict__ q_gain, const float* __restrict__ k_gain,
-                                         float eps, int unit, int* __restrict__ error) {
+                                         float eps, int unit, int whole, int v_from_k, int* __restrict__ error) {
     extern __shared__ __align__(32) float nr_smem[];   // [warps][dim]
+    __shared__ float scratch[32];
     constexpr int STEP = VEC ? 8 : 1;
     const int t = blockIdx.x;
     grid_dependency_wait();
@@ -1008,11 +1154,29 @@ __global__ void norm_rotate_write_kernel(T* __restrict__ proj, int ld, const int
     const int off = slot >= 0 ? slot % page_size : 0;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     float* mine = nr_smem + (size_t)warp * dim;
+    float whole_inv[2] = {1.f, 1.f};                   // of q, of k
+    if (whole) {
+#pragma unroll
+        for (int side = 0; side < 2; ++side) {
+            const T* src = row + (side ? (size_t)heads * dim : 0);
+            const int columns = (side ? kv_heads : heads) * dim;
+            float sq = 0.f;
+            for (int d = threadIdx.x * STEP; d < columns; d += blockDim.x * STEP) {
+                float v[8];
+                if (VEC) load8(src + d, v);
+                else v[0] = to_float(src[d]);
+#pragma unroll
+                for (int i = 0; i < STEP; ++i) sq += v[i] * v[i];
+            }
+            whole_inv[side] = 1.0f / sqrtf(block_sum(sq, scratch) / (float)columns + eps);
+        }
+    }
     for (int h = warp; h < heads + kv_heads; h += warps) {
         const bool is_q = h < heads;
         if (!is_q && slot < 0) continue;               // nothing to store (uniform over the warp)
         T* src = row + (size_t)h * dim;
         const float* gain = is_q ? q_gain : k_gain;
+        if (whole && gain) gain += (size_t)(is_q ? h : h - heads) * dim;
         float sq = 0.f;
         for (int d = lane * STEP; d < dim; d += 32 * STEP) {
             float v[8];
@@ -1024,7 +1188,7 @@ __global__ void norm_rotate_write_kernel(T* __restrict__ proj, int ld, const int
             else mine[d] = v[0];
         }
         if (gain || unit) {
-            const float inv = 1.0f / sqrtf(warp_sum(sq) / (float)dim + eps);
+            const float inv = whole ? whole_inv[is_q ? 0 : 1] : 1.0f / sqrtf(warp_sum(sq) / (float)dim + eps);
             // every lane changes what it wrote itself
             for (int d = lane * STEP; d < dim; d += 32 * STEP)
 #pragma unroll
@@ -1051,7 +1215,7 @@ __global__ void norm_rotate_write_kernel(T* __restrict__ proj, int ld, const int
         __syncwarp();
     }
     if (slot < 0) return;
-    const T* v = row + (size_t)(heads + kv_heads) * dim;
+    const T* v = row + (size_t)(v_from_k ? heads : heads + kv_heads) * dim;
     for (int e = threadIdx.x * STEP; e < kv_heads * vdim; e += blockDim.x * STEP) {
         const int g = e / vdim, d = e - g * vdim;
         T* dst = v_pages + page * page_stride + ((long long)g * page_size + off) * vdim + d;
@@ -1062,33 +1226,6 @@ __global__ void norm_rotate_write_kernel(T* __restrict__ proj, int ld, const int
         } else {
             *dst = v[e];
         }
-    }
-}
-
-// out[t, h, :] <- out[t, h, :] * sigmoid(gate[t, h]): one number per token and head.  VEC: vdim a
-// multiple of 8 and rows on 16 bytes, eight columns per thread and trip.
-template <typename T, bool VEC>
-__global__ void head_gate_kernel(T* __restrict__ out, int out_ld, const T* __restrict__ gate, int gate_ld,
-                                 int heads, int vdim) {
-    grid_dependency_wait();
-    grid_dependents_go();
-    const size_t t = blockIdx.x;
-    T* o = out + t * out_ld;
-    const T* g = gate + t * gate_ld;
-    if (VEC) {
-        for (int c = threadIdx.x * 8; c < heads * vdim; c += blockDim.x * 8) {
-            const float s = 1.0f / (1.0f + expf(-to_float(g[c / vdim])));
-            float v[8];
-            load8(o + c, v);
-#pragma unroll
-            for (int i = 0; i < 8; ++i) v[i] *= s;
-            store8(o + c, v);
-        }
-        return;
-    }
-    for (int c = threadIdx.x; c < heads * vdim; c += blockDim.x) {
-        const float s = 1.0f / (1.0f + expf(-to_float(g[c / vdim])));
-        o[c] = from_float<T>(to_float(o[c]) * s);
     }
 }
 
@@ -1141,28 +1278,37 @@ static int scaled_attention_rows_launch(const ScaledAttnParams& p, int tiles, bo
 
 template <bool FEW>
 static int scaled_attention_rows_dispatch(const ScaledAttnParams& p, int tiles, bool shared_v, cudaStream_t stream) {
-    switch (p.value_dim / 64) {
-        case 1: return scaled_attention_rows_launch<8, FEW>(p, tiles, shared_v, stream);
-        case 2: return scaled_attention_rows_launch<16, FEW>(p, tiles, shared_v, stream);
-        case 3: return scaled_attention_rows_launch<24, FEW>(p, tiles, shared_v, stream);
-        default: return scaled_attention_rows_launch<32, FEW>(p, tiles, shared_v, stream);
+    switch (p.value_dim / 32) {
+        case 1: return scaled_attention_rows_launch<4, FEW>(p, tiles, shared_v, stream);
+        case 2: return scaled_attention_rows_launch<8, FEW>(p, tiles, shared_v, stream);
+        case 3: return scaled_attention_rows_launch<12, FEW>(p, tiles, shared_v, stream);
+        case 4: return scaled_attention_rows_launch<16, FEW>(p, tiles, shared_v, stream);
+        case 6: return scaled_attention_rows_launch<24, FEW>(p, tiles, shared_v, stream);
+        case 8: return scaled_attention_rows_launch<32, FEW>(p, tiles, shared_v, stream);
+        default: return ERR_UNSUPPORTED;
     }
 }
 
-// whether the tensor-core form of a warp per 16 rows takes these sizes (value sizes up to 256)
+// whether the tensor-core form of a warp per 16 rows takes these sizes (values of 32, 64, 96, 128, 192 or 256)
 static bool scaled_attention_rows_takes(int key_dim, int value_dim, bool shared_v, bool few) {
-    return value_dim <= 256 && RowsLayout(key_dim, value_dim, shared_v, few).total <= 226 * 1024;
+    const bool columns = value_dim == 32 || value_dim == 64 || value_dim == 96 || value_dim == 128 ||
+                         value_dim == 192 || value_dim == 256;
+    return columns && key_dim % 16 == 0 && RowsLayout(key_dim, value_dim, shared_v, few).total <= 226 * 1024;
 }
 
-// whether the tensor-core form takes these sizes and addresses
+// whether the tensor-core forms take these addresses and row strides
+static bool scaled_attention_mma_aligned(const ScaledAttnParams& p) {
+    if (p.page_stride % 8 || p.q_ld % 8 || p.out_ld % 2 || p.value_ld % 8) return false;
+    if (((size_t)p.q | (size_t)p.k_pages | (size_t)p.v_pages) & 15 || ((size_t)p.out & 3) || p.q_dim % 8) return false;
+    return !(p.gate && (p.gate_ld % 2 || ((size_t)p.gate & 3)));
+}
+
+// whether the tensor-core form whose warps split the value columns takes these sizes and addresses
 static bool scaled_attention_mma_takes(const ScaledAttnParams& p, int dtype, bool shared_v) {
     const int dv = p.value_dim;
     if (dtype != DTYPE_BF16 || p.key_dim % 16 || !(dv == 64 || dv == 128 || dv == 192 || dv == 256 || dv == 384 || dv == 512))
         return false;
-    if (p.page_stride % 8 || p.q_ld % 8 || p.out_ld % 2 || p.value_ld % 8) return false;
-    if (((size_t)p.q | (size_t)p.k_pages | (size_t)p.v_pages) & 15 || ((size_t)p.out & 3)) return false;
-    if (p.gate && (p.gate_ld % 2 || ((size_t)p.gate & 3))) return false;
-    return MmaLayout(p.key_dim, dv, shared_v).total <= 227 * 1024;
+    return scaled_attention_mma_aligned(p) && MmaLayout(p.key_dim, dv, shared_v).total <= 227 * 1024;
 }
 
 }  // namespace fsie
@@ -1174,12 +1320,12 @@ extern "C" {
 int fsie_scaled_attention_rows() { return SA_ROWS; }
 
 // Query rows of one tile for these sizes: 64 where a warp of the tensor-core kernel owns 16 rows
-// with all their value columns (bfloat16, key sizes in steps of 16, value sizes 64, 128, 192, 256;
+// with all their value columns (bfloat16, key sizes in steps of 16, value sizes 32, 64, 96, 128, 192, 256;
 // form 0 or 2), else 32.  The caller cuts its tile list accordingly.  form 3 asks for the
 // tensor-core kernel whose warps split the value columns at any value size it takes, form 4 for the one
 // whose warps split the keys of a tile of up to 16 rows (16, or 0 where it does not take the sizes).
 int fsie_scaled_attention_tile_rows(int dtype, int key_dim, int value_dim, int values_in_keys, int form) {
-    const bool sizes = dtype == DTYPE_BF16 && key_dim % 16 == 0 && value_dim % 64 == 0;
+    const bool sizes = dtype == DTYPE_BF16 && key_dim % 16 == 0;
     if (form == 4)
         return sizes && scaled_attention_rows_takes(key_dim, value_dim, values_in_keys != 0, true) ? TR_FEW_ROWS : 0;
     if (!sizes || form == 1 || form == 3) return SA_ROWS;
@@ -1194,21 +1340,27 @@ int fsie_scaled_attention_tile_rows(int dtype, int key_dim, int value_dim, int v
 // [nsplit, tokens, heads, 2] (float); the ranges are merged after the launch.  softcap 0: no cap on
 // the scores; gate null, or heads x value_dim columns per token of the storage type, rows gate_ld apart.
 // combine_tokens null: every token's ranges are merged, else those of the num_combine tokens it lists.
+// head_gate null, or one number per head and token, rows head_gate_ld apart; sink null or [heads];
+// pos_scale null, or [pos_len] factors by the query's position; maps, partial: see the head of this file
+// (`heads` counts every map's query heads; with `partial` nothing is merged and `out` is not written).
 int fsie_scaled_attention(const void* q, int q_ld, const float* head_scale, const void* k_pages,
                           const void* v_pages, long long page_stride, int page_size, int key_dim,
                           int value_dim, int values_in_keys, const int* block_tables, int bt_stride,
                           const int* tile_item, const int* tile_row0, int tiles, const int* item_qstart,
                           const int* item_qlen, const int* item_pos0, const int* item_slots, void* out,
                           int out_ld, float* part_o, float* part_ml, int tokens, int heads, int kv_heads,
-                          int window, int chunk, float softcap, const void* gate, int gate_ld, int nsplit,
+                          int window, int chunk, float softcap, const void* gate, int gate_ld,
+                          const void* head_gate, int head_gate_ld, const float* sink, const float* pos_scale,
+                          int pos_len, int maps, int partial, int nsplit,
                           const int* combine_tokens, int num_combine, int dtype, int form, int* error,
                           cudaStream_t stream) {
     if (tokens <= 0 || tiles <= 0) return 0;
     if (tiles > 65535 || nsplit > 65535) return ERR_UNSUPPORTED;
     if (key_dim <= 0 || value_dim <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || nsplit < 1 ||
-        page_size <= 0 || window < 0 || chunk < 0 || !(softcap >= 0.f) || (values_in_keys && value_dim > key_dim))
+        page_size <= 0 || window < 0 || chunk < 0 || !(softcap >= 0.f) || (values_in_keys && value_dim > key_dim) ||
+        maps < 1 || key_dim % maps != 0 || heads % (kv_heads * maps) != 0 || (pos_scale && pos_len <= 0))
         return ERR_BAD_ARGUMENT;
-    if (nsplit > 1 && (!part_o || !part_ml)) return ERR_BAD_ARGUMENT;
+    if ((nsplit > 1 || partial) && (!part_o || !part_ml)) return ERR_BAD_ARGUMENT;
     ScaledAttnParams p;
     p.q = q; p.q_ld = q_ld; p.head_scale = head_scale;
     p.k_pages = k_pages; p.v_pages = values_in_keys ? k_pages : v_pages;
@@ -1220,6 +1372,8 @@ int fsie_scaled_attention(const void* q, int q_ld, const float* head_scale, cons
     p.out = out; p.out_ld = out_ld; p.part_o = part_o; p.part_ml = part_ml;
     p.tokens = tokens; p.heads = heads; p.kv_heads = kv_heads; p.window = window; p.nsplit = nsplit;
     p.chunk = chunk; p.softcap = softcap; p.gate = gate; p.gate_ld = gate_ld;
+    p.head_gate = head_gate; p.head_gate_ld = head_gate_ld; p.sink = sink;
+    p.pos_scale = pos_scale; p.pos_len = pos_len; p.maps = maps; p.q_dim = key_dim / maps; p.partial = partial;
     p.error = error;
     p.page_shift = -1;
     for (int b = 0; b < 30; ++b)
@@ -1229,7 +1383,7 @@ int fsie_scaled_attention(const void* q, int q_ld, const float* head_scale, cons
     if (tile_rows == 0) return ERR_UNSUPPORTED;
     if (tile_rows != SA_ROWS) {
         // the caller has cut tiles of 64 (or 16) rows: no other kernel may take them
-        if (!scaled_attention_mma_takes(p, dtype, values_in_keys != 0)) return ERR_UNSUPPORTED;
+        if (!scaled_attention_mma_aligned(p)) return ERR_UNSUPPORTED;
         rc = tile_rows == TR_ROWS ? scaled_attention_rows_dispatch<false>(p, tiles, values_in_keys != 0, stream)
                                   : scaled_attention_rows_dispatch<true>(p, tiles, values_in_keys != 0, stream);
     } else if (form != 1 && scaled_attention_mma_takes(p, dtype, values_in_keys != 0)) {
@@ -1247,16 +1401,45 @@ int fsie_scaled_attention(const void* q, int q_ld, const float* head_scale, cons
         rc = dtype == DTYPE_F32 ? scaled_attention_dispatch<float>(p, tiles, values_in_keys != 0, stream)
                                 : scaled_attention_dispatch<bf16>(p, tiles, values_in_keys != 0, stream);
     }
-    if (rc != 0 || nsplit == 1) return rc;
+    if (rc != 0 || nsplit == 1 || partial) return rc;
     const dim3 cgrid(combine_tokens ? num_combine : tokens, heads);
     if (cgrid.x == 0) return 0;
     const int threads = value_dim >= 128 ? 128 : (value_dim >= 64 ? 64 : 32);
     if (dtype == DTYPE_F32)
         return launch_dependent(sa_combine_kernel<float>, cgrid, dim3(threads), 0, stream, part_o, part_ml, (float*)out,
                                 out_ld, tokens, heads, value_dim, nsplit, (const float*)gate, gate_ld,
-                                combine_tokens);
+                                (const float*)head_gate, head_gate_ld, sink, combine_tokens);
     return launch_dependent(sa_combine_kernel<bf16>, cgrid, dim3(threads), 0, stream, part_o, part_ml, (bf16*)out,
-                            out_ld, tokens, heads, value_dim, nsplit, (const bf16*)gate, gate_ld, combine_tokens);
+                            out_ld, tokens, heads, value_dim, nsplit, (const bf16*)gate, gate_ld,
+                            (const bf16*)head_gate, head_gate_ld, sink, combine_tokens);
+}
+
+// Merges what fsie_scaled_attention or fsie_attn_tc_scaled left with `partial` for 2 x heads query heads
+// (map m of head h is query head 2 h + m): part_o [nsplit, tokens, 2 heads, value_dim], part_ml [nsplit,
+// tokens, 2 heads, 2].  out [tokens, out_ld] gets heads x value_dim columns; gate null, or one number per
+// head and token, rows gate_ld apart.  combine_tokens as in fsie_scaled_attention.
+int fsie_difference_merge(const float* part_o, const float* part_ml, void* out, int out_ld, int tokens, int heads,
+                          int value_dim, int nsplit, float lambda, float eps, float factor, const void* gate,
+                          int gate_ld, const int* combine_tokens, int num_combine, int dtype, cudaStream_t stream) {
+    const int count = combine_tokens ? num_combine : tokens;
+    if (count <= 0 || heads <= 0) return 0;
+    if (!part_o || !part_ml || !out || nsplit < 1 || value_dim <= 0) return ERR_BAD_ARGUMENT;
+    if (value_dim > 512) return ERR_UNSUPPORTED;
+    const int warps = 4;
+    const dim3 grid((unsigned)(((long long)count * heads + warps - 1) / warps));
+    const bool vec = value_dim % 4 == 0 && out_ld % 4 == 0 && ((size_t)part_o & 15) == 0 &&
+                     ((size_t)out & (dtype == DTYPE_F32 ? 15 : 7)) == 0;
+#define FSIE_DIFFERENCE(T, V, N)                                                                                   \
+    launch_dependent(difference_merge_kernel<T, V, N>, grid, dim3(32 * warps), 0, stream, part_o, part_ml, (T*)out, \
+                     out_ld, tokens, heads, value_dim, nsplit, lambda, eps, factor, (const T*)gate, gate_ld,        \
+                     combine_tokens, count)
+#define FSIE_DIFFERENCE_SIZE(T)                                                                      \
+    (vec ? (value_dim <= 128 ? FSIE_DIFFERENCE(T, 4, 1) : (value_dim <= 256 ? FSIE_DIFFERENCE(T, 4, 2) \
+                                                                            : FSIE_DIFFERENCE(T, 4, 4)))  \
+         : (value_dim <= 128 ? FSIE_DIFFERENCE(T, 1, 4) : FSIE_DIFFERENCE(T, 1, 16)))
+    return dtype == DTYPE_F32 ? FSIE_DIFFERENCE_SIZE(float) : FSIE_DIFFERENCE_SIZE(bf16);
+#undef FSIE_DIFFERENCE_SIZE
+#undef FSIE_DIFFERENCE
 }
 
 // proj [tokens, ld] = q | k | v head by head; cos_sin [table_len, rotary_dim]; slot_of [tokens]
@@ -1284,16 +1467,17 @@ int fsie_rotate_mix_write(void* proj, int ld, const int* positions, const float*
 
 
 // proj [tokens, ld] = q | k | v head by head (more columns may follow); q_gain / k_gain [dim] float or
-// null (no norm of that side, or - unit != 0 - a norm without a gain); cos_sin [table_len, rotary_dim]; slot_of [tokens] (page * page_size +
+// null (no norm of that side, or - unit != 0 - a norm without a gain; [heads * dim] and [kv_heads * dim]
+// with `whole`, which needs a gain or unit on both sides); v_from_k: q | k only; cos_sin [table_len, rotary_dim]; slot_of [tokens] (page * page_size +
 // offset, -1: store nothing).
 int fsie_norm_rotate_write(void* proj, int ld, const int* positions, const float* cos_sin, int table_len,
                            const int* slot_of, void* k_pages, void* v_pages, long long page_stride,
                            int page_size, int tokens, int heads, int kv_heads, int dim, int vdim,
                            int rotary_dim, const float* q_gain, const float* k_gain, float eps, int unit,
-                           int dtype, int* error, cudaStream_t stream) {
+                           int whole, int v_from_k, int dtype, int* error, cudaStream_t stream) {
     if (tokens <= 0) return 0;
-    if (rotary_dim < 0 || rotary_dim > dim || (rotary_dim & 1) || dim <= 0 ||
-        ld < (heads + kv_heads) * dim + kv_heads * vdim)
+    if (rotary_dim < 0 || rotary_dim > dim || (rotary_dim & 1) || dim <= 0 || (v_from_k && vdim != dim) ||
+        ld < (heads + kv_heads) * dim + (v_from_k ? 0 : kv_heads * vdim))
         return ERR_BAD_ARGUMENT;
     // a token's heads share a block; where tokens are few, a warp for each head
     const int warps = tokens <= 64 ? (heads + kv_heads < 16 ? heads + kv_heads : 16) : 8;
@@ -1307,23 +1491,10 @@ int fsie_norm_rotate_write(void* proj, int ld, const int* positions, const float
 #define FSIE_NORM_ROTATE(T, V)                                                                                      \
     launch_dependent(norm_rotate_write_kernel<T, V>, dim3(tokens), dim3(warps * 32), smem, stream, (T*)proj, ld,    \
                      positions, cos_sin, table_len, slot_of, (T*)k_pages, (T*)v_pages, page_stride, page_size,     \
-                     heads, kv_heads, dim, vdim, rotary_dim, q_gain, k_gain, eps, unit, error)
+                     heads, kv_heads, dim, vdim, rotary_dim, q_gain, k_gain, eps, unit, whole, v_from_k, error)
     if (dtype == DTYPE_F32) return vec ? FSIE_NORM_ROTATE(float, true) : FSIE_NORM_ROTATE(float, false);
     return vec ? FSIE_NORM_ROTATE(bf16, true) : FSIE_NORM_ROTATE(bf16, false);
 #undef FSIE_NORM_ROTATE
-}
-
-// out [tokens, out_ld] holds heads x vdim columns per token, gate [tokens, gate_ld] one column per head.
-int fsie_head_gate(void* out, int out_ld, const void* gate, int gate_ld, int tokens, int heads, int vdim,
-                   int dtype, cudaStream_t stream) {
-    if (tokens <= 0 || heads <= 0 || vdim <= 0) return 0;
-    const bool vec = vdim % 8 == 0 && out_ld % 8 == 0 && (((size_t)out) & (dtype == DTYPE_F32 ? 31 : 15)) == 0;
-    const int threads = vec ? (heads * vdim >= 2048 ? 256 : 128) : (heads * vdim >= 1024 ? 256 : 128);
-#define FSIE_HEAD_GATE(T, V) launch_dependent(head_gate_kernel<T, V>, dim3(tokens), dim3(threads), 0, stream, (T*)out, \
-                                              out_ld, (const T*)gate, gate_ld, heads, vdim)
-    if (dtype == DTYPE_F32) return vec ? FSIE_HEAD_GATE(float, true) : FSIE_HEAD_GATE(float, false);
-    return vec ? FSIE_HEAD_GATE(bf16, true) : FSIE_HEAD_GATE(bf16, false);
-#undef FSIE_HEAD_GATE
 }
 
 }  // extern "C"

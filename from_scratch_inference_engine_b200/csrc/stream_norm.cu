@@ -3,7 +3,8 @@
 // the next sublayer's input and norms it, in one pass over the token's streams:
 //
 //   settle     x_t <- sum_r mix[r, t] x_r + out[t] y      for all t at once, from the old streams
-//              (only with a pending output y; written back when write_x)
+//              (only with a pending output y; written back when write_x; with y_scale [width] the
+//              output is first multiplied by it column by column)
 //   gather     u = sum_t in[t] x_t                        (in = null: the plain sum)
 //   norm       centred: z = T( (u - mean) / sqrt(mean((u - mean)^2) + eps) * gain + bias )
 //              else:    z = T( u / sqrt(mean(u^2) + eps) * gain + bias )
@@ -20,6 +21,7 @@ struct StreamNormParams {
     float* x;                      // [tokens, streams, width]
     const float* start;            // [tokens, width] or null
     const void* y;                 // [tokens, width] of T, or null: nothing pending
+    const float* y_scale;          // [width], or null: y as it is
     const float* mix;              // [streams, streams], from x to
     const float* out;              // [streams]
     const float* in;               // [streams] or null
@@ -88,7 +90,14 @@ __global__ void __launch_bounds__(512, S > 0 && S <= 4 ? 2 : 1) stream_norm_kern
         for (int i = 0; i < STEP; ++i) acc[i] = 0.f;
         if (S > 0) {
             float old[S > 0 ? S : 1][STEP], y[STEP];
-            if (settle) load4(yr + c, y);
+            if (settle) {
+                load4(yr + c, y);
+                if (p.y_scale) {
+                    load4(p.y_scale + c, v);
+#pragma unroll
+                    for (int i = 0; i < STEP; ++i) y[i] *= v[i];
+                }
+            }
             if (sr) {
                 load4(sr + c, old[0]);
 #pragma unroll
@@ -125,7 +134,7 @@ __global__ void __launch_bounds__(512, S > 0 && S <= 4 ? 2 : 1) stream_norm_kern
                 float* mine = stash + threadIdx.x;
                 for (int a = 0; a < streams; ++a)
                     mine[a * blockDim.x] = sr ? sr[c + i] : xr[(size_t)a * width + c + i];
-                const float y = settle ? to_float(yr[c + i]) : 0.f;
+                const float y = settle ? to_float(yr[c + i]) * (p.y_scale ? p.y_scale[c + i] : 1.f) : 0.f;
                 for (int b = 0; b < streams; ++b) {
                     float nv = mine[b * blockDim.x];
                     if (settle) {
@@ -208,17 +217,17 @@ using namespace fsie;
 
 extern "C" {
 
-int fsie_stream_norm(float* x, const float* start, const void* y, const float* mix, const float* out,
+int fsie_stream_norm(float* x, const float* start, const void* y, const float* y_scale, const float* mix, const float* out,
                      const float* in, const float* gain, const float* bias, const int* rows, void* z,
                      int num_rows, int streams, int width, float eps, int write_x, int centred, int dtype,
                      cudaStream_t stream) {
     if (num_rows <= 0) return 0;
     if (streams <= 0 || width <= 0 || !x || (y && (!mix || !out)) || (z && !gain) || (!y && !z)) return ERR_BAD_ARGUMENT;
     StreamNormParams p;
-    p.x = x; p.start = start; p.y = y; p.mix = mix; p.out = out; p.in = in; p.gain = gain; p.bias = bias;
+    p.x = x; p.start = start; p.y = y; p.y_scale = y_scale; p.mix = mix; p.out = out; p.in = in; p.gain = gain; p.bias = bias;
     p.rows = rows; p.z = z; p.streams = streams; p.width = width; p.write_x = write_x; p.centred = centred;
     p.eps = eps;
-    const size_t wide = (size_t)x | (size_t)start | (size_t)gain | (size_t)bias;
+    const size_t wide = (size_t)x | (size_t)start | (size_t)gain | (size_t)bias | (size_t)y_scale;
     const size_t stored = (size_t)y | (size_t)z;
     const bool vec = width % 4 == 0 && (wide & 15) == 0 && (stored & (dtype == DTYPE_F32 ? 15 : 7)) == 0;
     if (dtype == DTYPE_F32)

@@ -135,19 +135,21 @@ class Runtime:
         return self._tables[key]
 
     def prepare_weight(self, weight: torch.Tensor, swiglu: bool = False,
-                       activation: str = "silu") -> None:
+                       activation: str = "silu", plain_activation: Optional[str] = None) -> None:
         """Called by a part at bind for a matrix it will multiply activations with.  Large
         bfloat16 matrices get a TMA descriptor for the tcgen05 product that steps of few
-        tokens use (the library product is kept where it measured faster: small matrices)."""
+        tokens use (the library product is kept where it measured faster: small matrices).
+        `plain_activation`: the weight is for `linear_activated` only."""
         if self.dtype is not torch.bfloat16 or weight.dtype is not torch.bfloat16:
             return
         rows, k = weight.shape
         if k % 8 or (swiglu and rows % 2):
             return
         if self.products == "own":
-            self._tiled_weights[weight.data_ptr()] = (weight, swiglu, activation)
+            self._tiled_weights[weight.data_ptr()] = (weight, swiglu, activation, plain_activation)
         if rows * k >= self.few_token_min_elements:
-            self._few_token_weights[weight.data_ptr()] = ops.DecodeWeight(weight, swiglu, activation)
+            self._few_token_weights[weight.data_ptr()] = ops.DecodeWeight(weight, swiglu, activation,
+                                                                          plain_activation)
 
     def _tiled(self, x: torch.Tensor, weight: torch.Tensor) -> Optional["ops.TiledWeight"]:
         """The weight's descriptor for the tiled product when this step is one for it: more
@@ -163,8 +165,7 @@ class Runtime:
         if ops.gemm_tiles_count(x.shape[0], n, swiglu) < least:
             return None
         if not known:
-            prepared = self._tiled_weights[weight.data_ptr()] = ops.TiledWeight(prepared[0], swiglu,
-                                                                                 prepared[2])
+            prepared = self._tiled_weights[weight.data_ptr()] = ops.TiledWeight(*prepared)
         return prepared
 
     def _tiled_product(self, prepared, x, bias, out_dtype, tag=None) -> torch.Tensor:
@@ -214,6 +215,23 @@ class Runtime:
         if bias is None:
             return torch.mm(x, weight.t(), out=out)
         return torch.addmm(bias, x, weight.t(), out=out)
+
+    def linear_activated(self, x: torch.Tensor, weight: torch.Tensor, activation: str,
+                         tag: Optional[str] = None) -> torch.Tensor:
+        """act(x @ weight.T) in the compute dtype, `activation` one of `ops.PLAIN_ACTIVATIONS`: in the
+        product's epilogue where the engine's own products take the step, else by a kernel behind it.
+        The weight was prepared with that `plain_activation`."""
+        if self.dtype is not torch.float32:
+            prepared = self._few_tokens(x, weight) or self._tiled(x, weight)
+            if isinstance(prepared, ops.DecodeWeight):
+                return self._few_token_product(prepared, x, None, torch.bfloat16, tag)
+            if prepared is not None:
+                return self._tiled_product(prepared, x, None, torch.bfloat16, tag)
+            if self._skinny(x, weight):
+                return ops.gemm_skinny(weight, x, self.buffer(tag, x.shape[0], weight.shape[0], torch.bfloat16), None,
+                                       plain_activation=activation)
+        # no kernel above takes the step, so neither does `linear` ask one of them for it
+        return ops.relu_squared(self.linear(x, weight, None, tag))
 
     def _skinny(self, x: torch.Tensor, weight: torch.Tensor) -> bool:
         """Whether the set-up-free product takes this step: few tokens, and a matrix that the

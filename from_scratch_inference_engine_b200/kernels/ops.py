@@ -18,6 +18,7 @@ from ..csrc import build
 DTYPE_F32, DTYPE_BF16 = 0, 1
 GATE_KINDS = {"silu": 0, "gelu_tanh": 1, "relu2": 2}   # activations of a feed-forward ("relu2": the square of relu)
 FUSED_GATES = ("silu", "gelu_tanh")        # ... those that the matrix products' gated epilogues know
+PLAIN_ACTIVATIONS = ("relu2",)             # ... and those that their plain epilogues know (no gate)
 
 
 class KernelError(RuntimeError):
@@ -385,7 +386,7 @@ def attn_tc(head_dim: int):
                                      i, i, i, i, i, i, f, p, i, p, p]
         lib.fsie_attn_tc_decode.argtypes = lib.fsie_attn_tc.argtypes
         lib.fsie_attn_tc_scaled.argtypes = [p, i, i, p, i, i, p, i, p, p, i, p, p, p, p, i, p, p,
-                                            i, i, i, i, i, i, p, i, f, p, i, p, i, p, p]
+                                            i, i, i, i, i, i, p, i, f, p, i, p, i, p, p, i, i, i, p, i, p, p]
         lib.fsie_attn_tc_decode_rows.argtypes = []
         for name in ("fsie_attn_tc_map_bytes", "fsie_attn_tc_pages_map", "fsie_attn_tc",
                      "fsie_attn_tc_scaled", "fsie_attn_tc_decode", "fsie_attn_tc_decode_rows"):
@@ -453,32 +454,57 @@ def attention_tc_scaled(pages_map: PagesMap, entry: int, q: torch.Tensor, q_ld: 
                         kv_heads: int, window: int, error: torch.Tensor, nsplit: int = 1,
                         part_o: Optional[torch.Tensor] = None, part_ml: Optional[torch.Tensor] = None,
                         chunk: int = 0, softcap: float = 0.0, gate: Optional[torch.Tensor] = None,
-                        combine_tokens: Optional[torch.Tensor] = None, num_combine: int = 0) -> torch.Tensor:
+                        combine_tokens: Optional[torch.Tensor] = None, num_combine: int = 0,
+                        head_gate: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None,
+                        pos_scale: Optional[torch.Tensor] = None, maps: int = 1,
+                        partial: bool = False) -> Optional[torch.Tensor]:
     """`scaled_attention` of prompt portions (bfloat16, keys and values as wide as `pages_map` says, tiles
     of `ATTENTION_TC_ROWS` query rows) with tcgen05.mma; the weights meet the values as two bfloat16
     halves.  `gate` rows and its first column start on 16 bytes."""
     _need(q, torch.bfloat16, "q", contiguous=False)
-    _need(out, torch.bfloat16, "out")
     _need(head_scale, torch.float32, "head_scale")
     head_dim = pages_map.head_dim
-    if head_scale.numel() != heads or out.numel() < tokens * heads * head_dim:
-        raise KernelError("attention_tc_scaled: shapes do not fit")
-    gate_ld = 0
-    if gate is not None:
-        _need(gate, torch.bfloat16, "gate", contiguous=False)
-        if gate.shape != (tokens, heads * head_dim) or gate.stride(1) != 1:
-            raise KernelError("attention_tc_scaled: gate is not of the result's shape")
-        gate_ld = gate.stride(0)
-    if nsplit > 1 and (part_o.numel() < nsplit * tokens * heads * head_dim or
+    gate_ld, head_gate_ld, pos_len = _scaled_attention_extras(
+        "attention_tc_scaled", q.dtype, head_scale, out, tokens, heads, head_dim, gate, head_gate, sink, pos_scale,
+        partial)
+    if (nsplit > 1 or partial) and (part_o.numel() < nsplit * tokens * heads * head_dim or
                        part_ml.numel() < nsplit * tokens * heads * 2):
         raise KernelError("attention_tc_scaled: split scratch is too small")
     _check(attn_tc(head_dim).fsie_attn_tc_scaled(
         pages_map.ptr, pages_map.entries, entry, _ptr(q), q_ld, pages_map.page_size, _ptr(block_tables),
         block_tables.stride(0), _ptr(tile_item), _ptr(tile_row0), num_tiles, _ptr(item_qstart), _ptr(item_qlen),
         _ptr(item_pos0), _ptr(out), heads * head_dim, _ptr(part_o), _ptr(part_ml), tokens, heads, kv_heads, head_dim,
-        window, nsplit, _ptr(head_scale), int(chunk), float(softcap), _ptr(gate), gate_ld, _ptr(combine_tokens),
+        window, nsplit, _ptr(head_scale), int(chunk), float(softcap), _ptr(gate), gate_ld, _ptr(head_gate),
+        head_gate_ld, _ptr(sink), _ptr(pos_scale), pos_len, int(maps), int(partial), _ptr(combine_tokens),
         num_combine, _ptr(error), _stream()), "attention_tc_scaled")
     return out
+
+
+def _scaled_attention_extras(what: str, dtype: torch.dtype, head_scale: torch.Tensor, out: Optional[torch.Tensor],
+                             tokens: int, heads: int, value_dim: int, gate: Optional[torch.Tensor],
+                             head_gate: Optional[torch.Tensor], sink: Optional[torch.Tensor],
+                             pos_scale: Optional[torch.Tensor], partial: bool) -> Tuple[int, int, int]:
+    """Checks of what the scaled attention kernels share; (row strides of the two gates, positions of
+    pos_scale)."""
+    if head_scale.numel() != heads:
+        raise KernelError(f"{what}: one scale per head is needed")
+    if not partial:
+        _need(out, dtype, "out")
+        if out.numel() < tokens * heads * value_dim:
+            raise KernelError(f"{what}: shapes do not fit")
+    for name, t, columns in (("gate", gate, heads * value_dim), ("head_gate", head_gate, heads)):
+        if t is not None:
+            _need(t, dtype, name, contiguous=False)
+            if t.shape != (tokens, columns) or t.stride(1) != 1:
+                raise KernelError(f"{what}: {name} must hold {columns} columns per token")
+    if sink is not None:
+        _need(sink, torch.float32, "sink")
+        if sink.numel() != heads:
+            raise KernelError(f"{what}: one sink per head is needed")
+    if pos_scale is not None:
+        _need(pos_scale, torch.float32, "pos_scale")
+    return (0 if gate is None else gate.stride(0), 0 if head_gate is None else head_gate.stride(0),
+            0 if pos_scale is None else pos_scale.numel())
 
 
 def attention_tc_decode(pages_map: PagesMap, entry: int, q: torch.Tensor, q_ld: int,
@@ -539,13 +565,27 @@ def gemm_decode_lib():
 GEMM_DECODE_MAX_TOKENS = 64
 
 
+def _epilogue(what: str, swiglu: bool, activation: str, plain_activation: Optional[str]) -> int:
+    """What a product's kernel is told about its epilogue: 0 plain, 1 and 2 a gate through SiLU or the tanh form
+    of GELU, 3 no gate and the square of relu on the result."""
+    if plain_activation is not None:
+        if swiglu or plain_activation not in PLAIN_ACTIVATIONS:
+            raise KernelError(f"{what}: without a gate the activation is one of {', '.join(PLAIN_ACTIVATIONS)}")
+        return 3
+    if swiglu and activation not in FUSED_GATES:
+        raise KernelError(f"{what}: the gate is one of {', '.join(FUSED_GATES)}")
+    return 1 + GATE_KINDS[activation] if swiglu else 0
+
+
 class DecodeWeight:
     """A bfloat16 weight [rows, K] prepared for `gemm_decode`: its TMA descriptor.
-    For SwiGLU the weight holds the gate rows and then as many up rows."""
+    For SwiGLU the weight holds the gate rows and then as many up rows; `plain_activation` ("relu2")
+    is applied to the result of a product without a gate."""
 
-    def __init__(self, weight: torch.Tensor, swiglu: bool = False, activation: str = "silu"):
+    def __init__(self, weight: torch.Tensor, swiglu: bool = False, activation: str = "silu",
+                 plain_activation: Optional[str] = None):
         _need(weight, torch.bfloat16, "weight")
-        self.gate = 1 + GATE_KINDS[activation] if swiglu else 0     # what the kernel is told
+        self.gate = _epilogue("gemm_decode", swiglu, activation, plain_activation)
         rows, k = weight.shape
         if k % 8:
             raise KernelError("gemm_decode: K must be a multiple of 8")
@@ -604,7 +644,7 @@ def gemm_skinny_lib():
     if _gemm_skinny is None:
         lib = build.load_library("gemm_skinny")
         i, ll, p = ctypes.c_int, ctypes.c_longlong, ctypes.c_void_p
-        lib.fsie_gemm_skinny.argtypes = [p, p, ll, p, ll, p, i, i, i, i, p]
+        lib.fsie_gemm_skinny.argtypes = [p, p, ll, p, ll, p, i, i, i, i, i, p]
         lib.fsie_gemm_skinny.restype = i
         lib.fsie_gemm_skinny_qkv_rope.argtypes = [p, p, ll, p, ll, p, i, i, p, p, i, p, p, p, ll, i,
                                                   i, i, i, p, p]
@@ -653,10 +693,10 @@ def gemm_skinny_qkv_rope(weight: torch.Tensor, x: torch.Tensor, out: torch.Tenso
 
 
 def gemm_skinny(weight: torch.Tensor, x: torch.Tensor, out: torch.Tensor,
-                bias: Optional[torch.Tensor]) -> torch.Tensor:
+                bias: Optional[torch.Tensor], plain_activation: Optional[str] = None) -> torch.Tensor:
     """out[T, N] = x[T, K] @ weight.T (+ bias) for T <= 16: no pipeline to fill, every lane asks
     for its weights straight from global memory (for matrices so small that set-up would
-    dominate).  out is bfloat16 or float32."""
+    dominate).  out is bfloat16 or float32.  `plain_activation` "relu2": the square of relu of the result."""
     gemm_skinny_lib()
     _need(weight, torch.bfloat16, "weight")
     _need(x, torch.bfloat16, "x", contiguous=False)
@@ -672,6 +712,7 @@ def gemm_skinny(weight: torch.Tensor, x: torch.Tensor, out: torch.Tensor,
         _need(bias, torch.bfloat16, "bias")
     _check(_gemm_skinny.fsie_gemm_skinny(_ptr(weight), _ptr(x), x.stride(0), _ptr(out), out.stride(0),
                                          _ptr(bias), tokens, n, k, int(out.dtype is torch.float32),
+                                         int(_epilogue("gemm_skinny", False, "silu", plain_activation) == 3),
                                          _stream()), "gemm_skinny")
     return out
 
@@ -708,11 +749,13 @@ def gemm_tiles_count(rows: int, n: int, swiglu: bool) -> int:
 
 class TiledWeight:
     """A bfloat16 weight [rows, K] prepared for `gemm_tiles`: its TMA descriptor (boxes of 128
-    rows).  For SwiGLU the weight holds the gate rows and then as many up rows."""
+    rows).  For SwiGLU the weight holds the gate rows and then as many up rows; `plain_activation`
+    ("relu2") is applied to the result of a product without a gate."""
 
-    def __init__(self, weight: torch.Tensor, swiglu: bool = False, activation: str = "silu"):
+    def __init__(self, weight: torch.Tensor, swiglu: bool = False, activation: str = "silu",
+                 plain_activation: Optional[str] = None):
         _need(weight, torch.bfloat16, "weight")
-        self.gate = 1 + GATE_KINDS[activation] if swiglu else 0     # what the kernel is told
+        self.gate = _epilogue("gemm_tiles", swiglu, activation, plain_activation)
         rows, k = weight.shape
         if k % 8:
             raise KernelError("gemm_tiles: K must be a multiple of 8")
@@ -755,7 +798,7 @@ def gemm_tiles(weight: TiledWeight, x: torch.Tensor, out: torch.Tensor,
         raise KernelError("gemm_tiles: x does not fit the weight (rows must start on 16 bytes)")
     if (out.shape[0] != rows or out.shape[1] != weight.n or out.stride(1) != 1
             or out.dtype not in (torch.bfloat16, torch.float32)
-            or (weight.swiglu and out.dtype is torch.float32)):
+            or (weight.gate and out.dtype is torch.float32)):
         raise KernelError("gemm_tiles: out does not fit")
     if bias is not None:
         _need(bias, torch.bfloat16, "bias")
@@ -784,13 +827,7 @@ class GroupedTiledWeight:
     def __init__(self, weight: torch.Tensor, swiglu: bool = False, activation: str = "silu",
                  plain_activation: Optional[str] = None):
         _need(weight, torch.bfloat16, "weight")
-        if swiglu and GATE_KINDS[activation] > 1:
-            raise KernelError("gemm_tiles_grouped: the gate is SiLU or the tanh form of GELU")
-        self.gate = 1 + GATE_KINDS[activation] if swiglu else 0
-        if plain_activation is not None:       # no gate: the activation on the product itself
-            if swiglu or plain_activation != "relu2":
-                raise KernelError("gemm_tiles_grouped: without a gate the activation is 'relu2'")
-            self.gate = 3
+        self.gate = _epilogue("gemm_tiles_grouped", swiglu, activation, plain_activation)
         groups, rows, k = weight.shape
         if k % 8 or (swiglu and rows % 2):
             raise KernelError("gemm_tiles_grouped: K must be a multiple of 8, a SwiGLU matrix hold "
@@ -891,7 +928,9 @@ def scan():
         lib = build.load_library("scan")
         i, f, ll, p = ctypes.c_int, ctypes.c_float, ctypes.c_longlong, ctypes.c_void_p
         lib.fsie_lightning_scan.argtypes = [p, i, i, i, i, p, p, p, i, p, p, p, i, i, i, p, p, i, i, p,
-                                            i, p, ll, p]
+                                            i, p, p, f, i, ll, p]
+        lib.fsie_row_decay.argtypes = [p, i, i, i, p, p, f, p, i, i, i, p]
+        lib.fsie_head_norm_silu.argtypes = [p, p, i, i, p, p, i, i, i, f, i, p]
         lib.fsie_silu_rows.argtypes = [p, i, i, p, i, i, p]
         lib.fsie_gated_rmsnorm.argtypes = [p, p, i, i, p, p, i, i, f, i, p]
         lib.fsie_ssd_max_taps.argtypes = []
@@ -899,7 +938,7 @@ def scan():
                                       p, i, i, p]
         lib.fsie_ssd_tails.argtypes = [p, i, i, p, p, p, i, p, ll, ll, i, i, i, p]
         lib.fsie_ssd_gate_norm.argtypes = [p, p, i, p, i, i, p, p, p, i, i, i, i, f, i, p]
-        for name in ("fsie_lightning_scan", "fsie_silu_rows", "fsie_gated_rmsnorm", "fsie_ssd_max_taps",
+        for name in ("fsie_lightning_scan", "fsie_row_decay", "fsie_head_norm_silu", "fsie_silu_rows", "fsie_gated_rmsnorm", "fsie_ssd_max_taps",
                      "fsie_ssd_prep", "fsie_ssd_tails", "fsie_ssd_gate_norm"):
             getattr(lib, name).restype = i
         _scan = lib
@@ -1007,21 +1046,23 @@ def lightning_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int,
                    heads: int, dim: int, vdim: int, seg_item: Optional[torch.Tensor] = None,
                    seg_row0: Optional[torch.Tensor] = None, num_segs: int = 0, seg_tokens: int = 0,
                    chunk_states: Optional[torch.Tensor] = None, share: int = 1,
-                   decay_tok: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   decay_tok: Optional[torch.Tensor] = None, decay_row: Optional[torch.Tensor] = None,
+                   out_scale: float = 1.0) -> torch.Tensor:
     """Per request and head, token by token: S = decay * S + k v^T, o = S^T q.  proj [tokens, ld]
     (float32) holds the ACTIVATED projections (`silu_rows`) at the given column offsets; state
     [slots, heads, dim, vdim] (float32; or [slots, n] with the heads' matrices in the first
     heads * dim * vdim floats of a slot) is read and left updated; out [tokens, heads * vdim]
     float32.  `decay_tok` (float32 [tokens, heads]) gives a decay per token and head in place of
-    `decay`; `share` heads in a row read the same q and k columns (q and k then hold heads / share
+    `decay`; `decay_row` (float32 [tokens, heads * dim]) one per token, head and state row - proj may then be
+    of either storage type; the outputs are multiplied by `out_scale`; `share` heads in a row read the same q and k columns (q and k then hold heads / share
     column groups of `dim`).
 
     With `seg_item` / `seg_row0` (int32, one entry per chunk of `seg_tokens` tokens, listed
     request by request) and `chunk_states` (float32, num_segs * heads * dim * vdim at least; with
-    `decay_tok` num_segs * heads more) the
+    `decay_tok` num_segs * heads more, with `decay_row` num_segs * heads * dim more) the
     chunks of long prompts run side by side: each sums its own tokens, the sums are chained into
     the state at every chunk's start, and each chunk runs again from there for its outputs."""
-    _need(proj, torch.float32, "proj")
+    _need(proj, torch.float32 if decay_row is None else None, "proj")
     _need(state, torch.float32, "state")
     if decay is not None:
         _need(decay, torch.float32, "decay")
@@ -1037,8 +1078,12 @@ def lightning_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int,
         _need(decay_tok, torch.float32, "decay_tok")
         if decay_tok.numel() < tokens * heads:
             raise KernelError("lightning_scan: decay_tok is too small")
+    elif decay_row is not None:
+        _need(decay_row, torch.float32, "decay_row")
+        if decay_row.numel() < tokens * heads * dim:
+            raise KernelError("lightning_scan: decay_row is too small")
     elif decay is None:
-        raise KernelError("lightning_scan: a decay per head or per token and head is needed")
+        raise KernelError("lightning_scan: a decay per head, per token and head or per state row is needed")
     state_stride = state.stride(0)
     if state_stride < heads * dim * vdim or (decay is not None and decay.numel() != heads):
         raise KernelError("lightning_scan: state or decay does not fit the heads")
@@ -1048,13 +1093,15 @@ def lightning_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int,
         _need(seg_item, torch.int32, "seg_item")
         _need(seg_row0, torch.int32, "seg_row0")
         _need(chunk_states, torch.float32, "chunk_states")
-        if chunk_states.numel() < num_segs * heads * (dim * vdim + (decay_tok is not None)):
+        kept = dim if decay_row is not None else int(decay_tok is not None)     # decays of a chunk, per head
+        if chunk_states.numel() < num_segs * heads * (dim * vdim + kept):
             raise KernelError("lightning_scan: chunk_states is too small")
     _check(scan().fsie_lightning_scan(_ptr(proj), ld, q_off, k_off, v_off, _ptr(item_qstart),
                                       _ptr(item_qlen), _ptr(item_slots), items, _ptr(state),
                                       _ptr(decay), _ptr(out), heads, dim, vdim, _ptr(seg_item),
                                       _ptr(seg_row0), num_segs, seg_tokens, _ptr(chunk_states),
-                                      int(share), _ptr(decay_tok), state_stride, _stream()),
+                                      int(share), _ptr(decay_tok), _ptr(decay_row), float(out_scale),
+                                      _tag(proj.dtype), state_stride, _stream()),
            "lightning_scan")
     return out
 
@@ -1139,6 +1186,39 @@ def ssd_gate_norm(o: torch.Tensor, act: torch.Tensor, proj: torch.Tensor, z_off:
     _check(scan().fsie_ssd_gate_norm(_ptr(o), _ptr(act), act.stride(0), _ptr(proj), proj.shape[1], z_off,
                                      _ptr(skip), _ptr(gain), _ptr(out), tokens, inner, vdim, int(parts),
                                      float(eps), _tag(proj.dtype), _stream()), "ssd_gate_norm")
+    return out
+
+
+def row_decay(proj: torch.Tensor, low_off: int, rank: int, weight_t: torch.Tensor, bias: torch.Tensor,
+              inv_tau: float, out: torch.Tensor) -> torch.Tensor:
+    """out[t, c] = sigmoid(sum_r proj[t, low_off + r] weight_t[r, c] + bias[c])^inv_tau, all in 32-bit:
+    weight_t [rank, columns], bias [columns] and out [tokens, columns] float32."""
+    _need(proj, None, "proj")
+    for name, t in (("weight_t", weight_t), ("bias", bias), ("out", out)):
+        _need(t, torch.float32, name)
+    tokens, ld = proj.shape
+    columns = bias.numel()
+    if weight_t.shape != (rank, columns) or low_off + rank > ld or out.numel() < tokens * columns:
+        raise KernelError("row_decay: shapes do not fit")
+    _check(scan().fsie_row_decay(_ptr(proj), ld, low_off, rank, _ptr(weight_t), _ptr(bias), float(inv_tau), _ptr(out),
+                                 tokens, columns, _tag(proj.dtype), _stream()), "row_decay")
+    return out
+
+
+def head_norm_silu(o: torch.Tensor, proj: torch.Tensor, g_off: int, gain: torch.Tensor, eps: float,
+                   out: torch.Tensor, heads: int) -> torch.Tensor:
+    """Head by head out = o / sqrt(mean(o^2) + eps) * gain * silu(proj[:, g_off + ...]): o float32 [tokens,
+    heads * vdim], gain float32 [vdim] shared by the heads."""
+    _need(o, torch.float32, "o")
+    _need(proj, None, "proj")
+    _need(gain, torch.float32, "gain")
+    _need(out, proj.dtype, "out")
+    tokens, width = o.shape
+    vdim = gain.numel()
+    if heads * vdim != width or g_off + width > proj.shape[1] or out.numel() < tokens * width:
+        raise KernelError("head_norm_silu: shapes do not fit")
+    _check(scan().fsie_head_norm_silu(_ptr(o), _ptr(proj), proj.shape[1], g_off, _ptr(gain), _ptr(out), tokens, heads,
+                                      vdim, float(eps), _tag(proj.dtype), _stream()), "head_norm_silu")
     return out
 
 
@@ -1337,10 +1417,11 @@ def mixers():
         lib.fsie_scaled_attention_tile_rows.argtypes = [i, i, i, i, i]
         lib.fsie_scaled_attention_tile_rows.restype = i
         lib.fsie_scaled_attention.argtypes = [p, i, p, p, p, ll, i, i, i, i, p, i, p, p, i, p, p, p, p,
-                                              p, i, p, p, i, i, i, i, i, f, p, i, i, p, i, i, i, p, p]
+                                              p, i, p, p, i, i, i, i, i, f, p, i, p, i, p, p, i, i, i, i, p, i, i, i, p, p]
+        lib.fsie_difference_merge.argtypes = [p, p, p, i, i, i, i, i, f, f, f, p, i, p, i, i, p]
         lib.fsie_norm_rotate_write.argtypes = [p, i, p, p, i, p, p, p, ll, i, i, i, i, i, i, i, p, p, f,
-                                               i, i, p, p]
-        lib.fsie_head_gate.argtypes = [p, i, p, i, i, i, i, i, p]
+                                               i, i, i, i, p, p]
+        lib.fsie_relu_squared.argtypes = [p, ll, i, p]
         lib.fsie_scaled_sum_rmsnorm.argtypes = [p, p, f, p, f, p, p, p, i, i, f, i, i, p]
         lib.fsie_rotate_mix_write.argtypes = [p, i, p, p, i, p, p, p, ll, i, i, i, i, i, i, i, i, p, p,
                                               i, p, p]
@@ -1348,8 +1429,8 @@ def mixers():
         lib.fsie_head_product.argtypes = [p, ll, i, p, p, ll, i, i, i, i, i, i, p]
         for name in ("fsie_norm_add_norm", "fsie_gated_act", "fsie_mingru_scan",
                      "fsie_scaled_attention_rows", "fsie_scaled_attention", "fsie_rotate_mix_write",
-                     "fsie_latent_prep", "fsie_head_product", "fsie_norm_rotate_write", "fsie_head_gate",
-                     "fsie_scaled_sum_rmsnorm"):
+                     "fsie_latent_prep", "fsie_head_product", "fsie_norm_rotate_write",
+                     "fsie_difference_merge", "fsie_relu_squared", "fsie_scaled_sum_rmsnorm"):
             getattr(lib, name).restype = i
         _mixers = lib
     return _mixers
@@ -1404,6 +1485,13 @@ def gated_act(gate_up: torch.Tensor, out: torch.Tensor, kind: str) -> torch.Tens
     return out
 
 
+def relu_squared(x: torch.Tensor) -> torch.Tensor:
+    """x <- relu(x)^2 in place (behind products whose kernel has no such epilogue)."""
+    _need(x, None, "x")
+    _check(mixers().fsie_relu_squared(_ptr(x), x.numel(), _tag(x.dtype), _stream()), "relu_squared")
+    return x
+
+
 def mingru_scan(proj: torch.Tensor, width: int, item_qstart: torch.Tensor, item_qlen: torch.Tensor,
                 item_slots: torch.Tensor, items: int, state: torch.Tensor, out: torch.Tensor,
                 seg_item: Optional[torch.Tensor] = None, seg_row0: Optional[torch.Tensor] = None,
@@ -1448,39 +1536,41 @@ def scaled_attention(q: torch.Tensor, q_ld: int, head_scale: torch.Tensor, k_pag
                      value_dim: int, values_in_keys: bool, block_tables: torch.Tensor,
                      tile_item: torch.Tensor, tile_row0: torch.Tensor, tiles: int,
                      item_qstart: torch.Tensor, item_qlen: torch.Tensor, item_pos0: torch.Tensor,
-                     item_slots: Optional[torch.Tensor], out: torch.Tensor, tokens: int, heads: int,
+                     item_slots: Optional[torch.Tensor], out: Optional[torch.Tensor], tokens: int, heads: int,
                      kv_heads: int, window: int, error: torch.Tensor, nsplit: int = 1,
                      part_o: Optional[torch.Tensor] = None,
                      part_ml: Optional[torch.Tensor] = None, form: str = "auto",
                      chunk: int = 0, softcap: float = 0.0, gate: Optional[torch.Tensor] = None,
-                     combine_tokens: Optional[torch.Tensor] = None, num_combine: int = 0) -> torch.Tensor:
+                     combine_tokens: Optional[torch.Tensor] = None, num_combine: int = 0,
+                     head_gate: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None,
+                     pos_scale: Optional[torch.Tensor] = None, maps: int = 1,
+                     partial: bool = False) -> Optional[torch.Tensor]:
     """Causal (optionally windowed; `chunk` > 0: only over the keys j with j // chunk == i // chunk)
     softmax attention of q [tokens, heads x key_dim] over paged keys
     [kv_head][slot][key_dim] and values [kv_head][slot][value_dim] (or, values_in_keys, the first
     value_dim columns of the key rows), scores multiplied by head_scale[head] and - `softcap` > 0 -
     passed through softcap * tanh(. / softcap); scores, softmax and weights in 32-bit.  `gate`
     [tokens, heads x value_dim] (may be a view of columns of a wider tensor): the result is multiplied
-    by its sigmoid column by column before it is rounded.  `combine_tokens` (int32, `num_combine` of them): the tokens
+    by its sigmoid column by column before it is rounded; `head_gate` [tokens, heads] by one sigmoid per
+    head.  `sink` (float32 [heads]): the denominator of a head's softmax also holds e^sink.  `pos_scale`
+    (float32): a factor on the scores of the query at each position.  `maps` > 1: a key row is that many
+    keys side by side, and query head h - `heads` counts them for every map, each key_dim / maps wide -
+    reads key h % maps of its key/value head.  `partial`: every key range's maximum, sum and unnormalised
+    output stay in part_o and part_ml (`difference_merge` takes them from there); `out` may be None.  `combine_tokens` (int32, `num_combine` of them): the tokens
     that the tiles hold, where they are not all the step's tokens (split ranges of others are not
     merged).  `form`: "auto" takes a tensor-core kernel where one fits (bfloat16, key
-    sizes in steps of 16, value sizes 64 ... 512), "plain" the 32-bit kernel, "mma" insists on a
+    sizes in steps of 16, value sizes 32 ... 512), "plain" the 32-bit kernel, "mma" insists on a
     tensor-core kernel, "mma_split" on the one whose warps split the value columns, "mma_few" on
     the one for tiles of up to 16 rows whose warps split a tile's keys.  The tiles
     hold `scaled_attention_rows(dtype, key_dim, value_dim, values_in_keys, form)` rows."""
     _need(q, None, "q", contiguous=False)
     _need(head_scale, torch.float32, "head_scale")
-    _need(out, q.dtype, "out")
     if k_pages.dtype is not q.dtype:
         raise KernelError("scaled_attention: cache dtype differs from q")
-    if head_scale.numel() != heads or out.numel() < tokens * heads * value_dim:
-        raise KernelError("scaled_attention: shapes do not fit")
-    gate_ld = 0
-    if gate is not None:
-        _need(gate, q.dtype, "gate", contiguous=False)
-        if gate.shape != (tokens, heads * value_dim) or gate.stride(1) != 1:
-            raise KernelError("scaled_attention: gate is not of the result's shape")
-        gate_ld = gate.stride(0)
-    if nsplit > 1:
+    gate_ld, head_gate_ld, pos_len = _scaled_attention_extras(
+        "scaled_attention", q.dtype, head_scale, out, tokens, heads, value_dim, gate, head_gate, sink, pos_scale,
+        partial)
+    if nsplit > 1 or partial:
         if part_o.numel() < nsplit * tokens * heads * value_dim or \
                 part_ml.numel() < nsplit * tokens * heads * 2:
             raise KernelError("scaled_attention: scratch for the key splits is too small")
@@ -1489,8 +1579,33 @@ def scaled_attention(q: torch.Tensor, q_ld: int, head_scale: torch.Tensor, k_pag
         value_dim, int(values_in_keys), _ptr(block_tables), block_tables.stride(0), _ptr(tile_item),
         _ptr(tile_row0), tiles, _ptr(item_qstart), _ptr(item_qlen), _ptr(item_pos0), _ptr(item_slots),
         _ptr(out), heads * value_dim, _ptr(part_o), _ptr(part_ml), tokens, heads, kv_heads, window,
-        int(chunk), float(softcap), _ptr(gate), gate_ld, nsplit, _ptr(combine_tokens), num_combine, _tag(q.dtype), SCALED_ATTENTION_FORMS[form], _ptr(error), _stream()),
-        "scaled_attention")
+        int(chunk), float(softcap), _ptr(gate), gate_ld, _ptr(head_gate), head_gate_ld, _ptr(sink), _ptr(pos_scale),
+        pos_len, int(maps), int(partial), nsplit, _ptr(combine_tokens), num_combine, _tag(q.dtype),
+        SCALED_ATTENTION_FORMS[form], _ptr(error), _stream()), "scaled_attention")
+    return out
+
+
+def difference_merge(part_o: torch.Tensor, part_ml: torch.Tensor, out: torch.Tensor, tokens: int, heads: int,
+                     value_dim: int, nsplit: int, weight: float, eps: float, factor: float,
+                     gate: Optional[torch.Tensor] = None, combine_tokens: Optional[torch.Tensor] = None,
+                     num_combine: int = 0) -> torch.Tensor:
+    """out[t, h] = o / sqrt(mean(o^2) + eps) * factor * sigmoid(gate[t, h]) with o = a_1 - weight * a_2, the
+    results of query heads 2 h and 2 h + 1 that a `partial` attention left in part_o [nsplit, tokens, 2
+    heads, value_dim] and part_ml [nsplit, tokens, 2 heads, 2] (float32), all in 32-bit."""
+    _need(part_o, torch.float32, "part_o")
+    _need(part_ml, torch.float32, "part_ml")
+    _need(out, None, "out")
+    if part_o.numel() < nsplit * tokens * 2 * heads * value_dim or part_ml.numel() < nsplit * tokens * 4 * heads or \
+            out.numel() < tokens * heads * value_dim:
+        raise KernelError("difference_merge: shapes do not fit")
+    if gate is not None:
+        _need(gate, out.dtype, "gate", contiguous=False)
+        if gate.shape != (tokens, heads) or gate.stride(1) != 1:
+            raise KernelError("difference_merge: gate must hold one number per head and token")
+    _check(mixers().fsie_difference_merge(
+        _ptr(part_o), _ptr(part_ml), _ptr(out), heads * value_dim, tokens, heads, value_dim, nsplit, float(weight),
+        float(eps), float(factor), _ptr(gate), 0 if gate is None else gate.stride(0), _ptr(combine_tokens), num_combine,
+        _tag(out.dtype), _stream()), "difference_merge")
     return out
 
 
@@ -1528,12 +1643,15 @@ def norm_rotate_write(proj: torch.Tensor, positions: torch.Tensor, cos_sin: torc
                       slot_of: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
                       page_stride: int, page_size: int, heads: int, kv_heads: int, dim: int, vdim: int,
                       rotary_dim: int, q_gain: Optional[torch.Tensor], k_gain: Optional[torch.Tensor],
-                      eps: float, error: torch.Tensor, unit: bool = False) -> None:
+                      eps: float, error: torch.Tensor, unit: bool = False, whole: bool = False,
+                      values_from_keys: bool = False) -> None:
     """proj [tokens, q | k | v | ...]: every head of q (of k) divided by its root mean square (eps
     inside the root) times q_gain (k_gain) [dim] in 32-bit where that gain is given (`unit`: where it is
-    not given, divided by its root mean square alone); then q rotated in
+    not given, divided by its root mean square alone; `whole`: the root mean square is over all heads of q
+    (of k) at once, the gains hold a number per column of all heads); then q rotated in
     place and k into its page over the first rotary_dim of each head (pairs i, i + rotary_dim / 2);
-    values into their page."""
+    values into their page (`values_from_keys`: proj holds no v, the values are the keys as projected,
+    before norm and rotation)."""
     _need(proj, None, "proj")
     _need(positions, torch.int32, "positions")
     _need(cos_sin, torch.float32, "cos_sin")
@@ -1543,29 +1661,20 @@ def norm_rotate_write(proj: torch.Tensor, positions: torch.Tensor, cos_sin: torc
         raise KernelError("norm_rotate_write: cos/sin table width differs from rotary_dim")
     if k_pages.dtype is not proj.dtype or v_pages.dtype is not proj.dtype:
         raise KernelError("norm_rotate_write: cache dtype differs from the projection dtype")
-    for name, gain in (("q_gain", q_gain), ("k_gain", k_gain)):
+    for name, gain, count in (("q_gain", q_gain, heads), ("k_gain", k_gain, kv_heads)):
         if gain is not None:
             _need(gain, torch.float32, name)
-            if gain.numel() != dim:
-                raise KernelError(f"norm_rotate_write: {name} must hold one number per column of a head")
+            if gain.numel() != (dim * count if whole else dim):
+                raise KernelError(f"norm_rotate_write: {name} must hold one number per column of "
+                                  f"{'all heads' if whole else 'a head'}")
+    if values_from_keys and vdim != dim:
+        raise KernelError("norm_rotate_write: values that are the keys are as wide as the keys")
     _check(mixers().fsie_norm_rotate_write(_ptr(proj), ld, _ptr(positions), _ptr(cos_sin), cos_sin.shape[0],
                                            _ptr(slot_of), _ptr(k_pages), _ptr(v_pages), page_stride,
                                            page_size, tokens, heads, kv_heads, dim, vdim, rotary_dim,
-                                           _ptr(q_gain), _ptr(k_gain), float(eps), int(unit),
+                                           _ptr(q_gain), _ptr(k_gain), float(eps), int(unit), int(whole),
+                                           int(values_from_keys),
                                            _tag(proj.dtype), _ptr(error), _stream()), "norm_rotate_write")
-
-
-def head_gate(out: torch.Tensor, gate: torch.Tensor, heads: int, vdim: int) -> torch.Tensor:
-    """out[t, h, :] <- out[t, h, :] * sigmoid(gate[t, h]); out [tokens, heads * vdim], `gate`
-    [tokens, heads] may be a view of columns of a wider tensor."""
-    _need(out, None, "out", contiguous=False)
-    _need(gate, out.dtype, "gate", contiguous=False)
-    tokens = out.shape[0]
-    if out.shape[1] != heads * vdim or gate.shape != (tokens, heads) or out.stride(1) != 1 or gate.stride(1) != 1:
-        raise KernelError("head_gate: shapes do not fit")
-    _check(mixers().fsie_head_gate(_ptr(out), out.stride(0), _ptr(gate), gate.stride(0), tokens, heads, vdim,
-                                   _tag(out.dtype), _stream()), "head_gate")
-    return out
 
 
 def scaled_sum_rmsnorm(x: torch.Tensor, deltas, scales, gain: Optional[torch.Tensor], eps: float,
@@ -1915,7 +2024,7 @@ def streams_lib():
     if _streams is None:
         lib = build.load_library("streams")
         i, f, p = ctypes.c_int, ctypes.c_float, ctypes.c_void_p
-        lib.fsie_stream_norm.argtypes = [p, p, p, p, p, p, p, p, p, p, i, i, i, f, i, i, i, p]
+        lib.fsie_stream_norm.argtypes = [p, p, p, p, p, p, p, p, p, p, p, i, i, i, f, i, i, i, p]
         lib.fsie_stream_norm.restype = i
         _streams = lib
     return _streams
@@ -1925,10 +2034,10 @@ def stream_norm(x: torch.Tensor, start: Optional[torch.Tensor], delta: Optional[
                 mix: Optional[torch.Tensor], spread: Optional[torch.Tensor], gather: Optional[torch.Tensor],
                 gain: Optional[torch.Tensor], bias: Optional[torch.Tensor], eps: float,
                 out: Optional[torch.Tensor], rows: Optional[torch.Tensor] = None, write_x: bool = True,
-                centred: bool = True) -> Optional[torch.Tensor]:
+                centred: bool = True, delta_scale: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """x (float32 [tokens, streams, width]) holds a token's streams; with `start` (float32 [tokens,
     width]) they do not exist yet and every one equals the token's row of it.  A pending sublayer
-    output `delta` [tokens, width] settles first: x_t <- sum_r mix[r, t] x_r + spread[t] delta for all
+    output `delta` [tokens, width] (times `delta_scale`, float32 [width], where given) settles first: x_t <- sum_r mix[r, t] x_r + spread[t] delta for all
     streams at once (mix [streams, streams], spread [streams], float32).  Then out = norm of
     sum_t gather[t] x_t (gather None: the plain sum), `centred` a layer norm (gain, bias), else an RMS
     norm, in out's dtype.  Without `out` only the settling.  With `rows` (int32 indices) only those
@@ -1948,6 +2057,10 @@ def stream_norm(x: torch.Tensor, start: Optional[torch.Tensor], delta: Optional[
         _need(spread, torch.float32, "spread")
         if delta.shape != (tokens, width) or mix.shape != (streams, streams) or spread.numel() != streams:
             raise KernelError("stream_norm: the pending output or its coefficients do not fit")
+        if delta_scale is not None:
+            _need(delta_scale, torch.float32, "delta_scale")
+            if delta_scale.numel() != width:
+                raise KernelError("stream_norm: one scale per column of the pending output")
     if gather is not None:
         _need(gather, torch.float32, "gather")
         if gather.numel() != streams:
@@ -1963,7 +2076,7 @@ def stream_norm(x: torch.Tensor, start: Optional[torch.Tensor], delta: Optional[
             _need(bias, torch.float32, "bias")
         if gain.numel() != width or (bias is not None and bias.numel() != width) or out.numel() < count * width:
             raise KernelError("stream_norm: gain, bias or out does not fit")
-    _check(streams_lib().fsie_stream_norm(_ptr(x), _ptr(start), _ptr(delta), _ptr(mix), _ptr(spread), _ptr(gather),
+    _check(streams_lib().fsie_stream_norm(_ptr(x), _ptr(start), _ptr(delta), _ptr(delta_scale), _ptr(mix), _ptr(spread), _ptr(gather),
                                           _ptr(gain), _ptr(bias), _ptr(rows), _ptr(out), count, streams, width,
                                           float(eps), int(write_x), int(centred), _tag(dtype), _stream()),
            "stream_norm")

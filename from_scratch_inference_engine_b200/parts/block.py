@@ -258,20 +258,27 @@ class ParallelBlock(Part):
 
 class _StreamCoefficients:
     """How one sublayer meets a residual of several streams: its input is sum_t gather[t] x_t, and its
-    output y changes every stream, x_t <- sum_r mix[r, t] x_r + spread[t] y."""
+    output y changes every stream, x_t <- sum_r mix[r, t] x_r + spread[t] y; with `scale_name` y is first
+    multiplied by that tensor column by column."""
 
-    def __init__(self, prefix: str, streams: int, names):
-        self.streams = streams
+    def __init__(self, prefix: str, streams: int, names, width: int, scale_name: Optional[str] = None):
+        self.streams, self.width = streams, width
         self.names = {which: prefix + name for which, name in names.items()}
-        self.gather = self.mix = self.spread = None
+        self.scale_name = None if scale_name is None else prefix + scale_name
+        self.gather = self.mix = self.spread = self.scale = None
 
     def tensor_specs(self, optional: bool = False) -> List[TensorSpec]:
         s = self.streams
-        return [TensorSpec(self.names["gather"], (s,), role="vector", init="gain", optional=optional),
-                TensorSpec(self.names["spread"], (s,), role="vector", init="gain", optional=optional),
-                TensorSpec(self.names["mix"], (s, s), role="vector", init="eye", optional=optional)]
+        specs = [TensorSpec(self.names["gather"], (s,), role="vector", init="gain", optional=optional),
+                 TensorSpec(self.names["spread"], (s,), role="vector", init="gain", optional=optional),
+                 TensorSpec(self.names["mix"], (s, s), role="vector", init="eye", optional=optional)]
+        if self.scale_name is not None:
+            specs.append(TensorSpec(self.scale_name, (self.width,), role="vector", init="gain", optional=optional))
+        return specs
 
     def bind(self, tensors) -> None:
+        if self.scale_name is not None:
+            self.scale = tensors[self.scale_name].to(torch.float32).contiguous()
         for which, name in self.names.items():
             setattr(self, which, tensors[name].to(torch.float32).contiguous())
 
@@ -287,7 +294,8 @@ class StreamsBlock(Part):
     next sublayer's, or the model's final norm on the wanted rows only - spreads it, gathers the
     streams and norms the gathered row in one pass.  The coefficients of sublayer q (1: mixer, 2:
     feed-forward) are the tensors "hc<q>.in", "hc<q>.out" and "hc<q>.mix" below the layer's prefix;
-    `STREAM_NAMES` names them.
+    `STREAM_NAMES` names them.  With the layer's `output_scale_names` (one per sublayer) every output is
+    multiplied by that tensor column by column before it is spread, in the same kernel.
     """
 
     STREAM_NAMES = ({"gather": "hc1.in", "spread": "hc1.out", "mix": "hc1.mix"},
@@ -300,8 +308,10 @@ class StreamsBlock(Part):
         self.mixer_norm = build_part("norm", layer.mixer_norm, prefix + layer.mixer_norm_name)
         self.mixer = build_part("mixer", layer.mixer, prefix + layer.mixer_name)
         self.feed_forward = self.feed_forward_norm = None
-        self.coefficients = [_StreamCoefficients(prefix, self.streams, self.STREAM_NAMES[0])]
-        second = _StreamCoefficients(prefix, self.streams, self.STREAM_NAMES[1])
+        scale_names = layer.output_scale_names or (None, None)
+        first, second = (_StreamCoefficients(prefix, self.streams, names, self.mixer_norm.width, scale_name)
+                         for names, scale_name in zip(self.STREAM_NAMES, scale_names))
+        self.coefficients = [first]
         # a checkpoint may still hold the norm and the coefficients of a feed-forward that the layer
         # does not have
         self.unused: List[TensorSpec] = []
@@ -347,9 +357,9 @@ class StreamsBlock(Part):
         y = self.mixer_norm.over_streams(x, delta, first.gather, tag="streams.mixer_in")
         # until an output has settled, the streams are the rows they all start from
         start = delta.start if delta.delta is None else None
-        delta = StreamUpdate(self.mixer.forward(ctx, y, cache), first.mix, first.spread, start)
+        delta = StreamUpdate(self.mixer.forward(ctx, y, cache), first.mix, first.spread, start, first.scale)
         if self.feed_forward is None:
             return delta
         second = self.coefficients[1]
         y = self.feed_forward_norm.over_streams(x, delta, second.gather, tag="streams.feed_forward_in")
-        return StreamUpdate(self.feed_forward.forward(ctx, y), second.mix, second.spread)
+        return StreamUpdate(self.feed_forward.forward(ctx, y), second.mix, second.spread, scale=second.scale)

@@ -1,4 +1,4 @@
-"""Dense gated feed-forward (SwiGLU, or another activation on the gate)."""
+"""Dense feed-forwards: gated (SwiGLU, or another activation on the gate), and without a gate."""
 
 from __future__ import annotations
 
@@ -73,3 +73,40 @@ class SwiGluMlp(Part):
         act = rt.linear_swiglu(y, self.w_gate_up, "swiglu.act", bias=self.b_gate_up,
                                activation=self.activation)
         return rt.linear(act, self.w_down, self.b_down, "swiglu.down")
+
+
+@register_part("feed_forward", "plain_mlp")
+class PlainMlp(Part):
+    """down( act(up(y)) ) without gate and biases, act one of `ops.PLAIN_ACTIVATIONS` ("relu2": the square
+    of relu), in the epilogue of the first product where the engine's own products take the step.
+    `names` gives the tensor names below the prefix."""
+
+    capturable = True
+
+    NAMES = {"up": "up", "down": "down"}
+
+    def __init__(self, prefix: str, hidden_size: int, intermediate_size: int, activation: str,
+                 names: Optional[Dict[str, str]] = None):
+        if activation not in ops.PLAIN_ACTIVATIONS:
+            raise ValueError(f"unknown activation '{activation}' ({', '.join(ops.PLAIN_ACTIVATIONS)})")
+        self.prefix, self.hidden_size = prefix, int(hidden_size)
+        self.intermediate_size, self.activation = int(intermediate_size), activation
+        self.names = dict(self.NAMES)
+        self.names.update(names or {})
+        self.w_up = self.w_down = None
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        h, i = self.hidden_size, self.intermediate_size
+        return [TensorSpec(self.prefix + self.names["up"], (i, h)),
+                TensorSpec(self.prefix + self.names["down"], (h, i))]
+
+    def bind(self, tensors: Dict[str, torch.Tensor], runtime) -> None:
+        self.runtime = runtime
+        self.w_up = tensors[self.prefix + self.names["up"]].contiguous()
+        self.w_down = tensors[self.prefix + self.names["down"]].contiguous()
+        runtime.prepare_weight(self.w_up, plain_activation=self.activation)
+        runtime.prepare_weight(self.w_down)
+
+    def forward(self, ctx, y: torch.Tensor) -> torch.Tensor:
+        act = self.runtime.linear_activated(y, self.w_up, self.activation, "plain_mlp.act")
+        return self.runtime.linear(act, self.w_down, None, "plain_mlp.down")

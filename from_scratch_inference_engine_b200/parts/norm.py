@@ -47,12 +47,13 @@ class StreamUpdate:
     """What is still to happen to a residual of several streams before the next sublayer reads it.
     `start` (float32 [tokens, width]): the streams do not exist yet, every one equals these rows.
     `delta`: a sublayer's output that is to be spread over the streams, x_t <- sum_r mix[r, t] x_r +
-    spread[t] delta (None: no sublayer has run)."""
+    spread[t] (scale * delta) (None: no sublayer has run), `scale` a number per column or None."""
 
     delta: Optional[torch.Tensor] = None
     mix: Optional[torch.Tensor] = None          # float32 [streams, streams], from x to
     spread: Optional[torch.Tensor] = None       # float32 [streams]
     start: Optional[torch.Tensor] = None
+    scale: Optional[torch.Tensor] = None        # float32 [width]
 
 
 class StreamNorm:
@@ -70,7 +71,8 @@ class StreamNorm:
         count = x.shape[0] if rows is None else rows.numel()
         out = self.runtime.buffer(tag, count, self.width, self.runtime.dtype)
         return ops.stream_norm(x, pending.start, pending.delta, pending.mix, pending.spread, gather, gain, bias,
-                               self.eps, out, rows=rows, write_x=write_x, centred=self.centred)
+                               self.eps, out, rows=rows, write_x=write_x, centred=self.centred,
+                               delta_scale=pending.scale)
 
 
 @register_part("norm", "rmsnorm")

@@ -33,12 +33,19 @@ def key_splits(blocks: int, longest: int, sms: int, key_tile: int = 32) -> int:
 def attend(ctx, rt, q: torch.Tensor, head_scale: torch.Tensor, group, cache: LayerCache,
            out: torch.Tensor, heads: int, kv_heads: int, key_dim: int, value_dim: int,
            values_in_keys: bool, window: int, chunk: int = 0, softcap: float = 0.0,
-           gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+           gate: Optional[torch.Tensor] = None, head_gate: Optional[torch.Tensor] = None,
+           sink: Optional[torch.Tensor] = None, pos_scale: Optional[torch.Tensor] = None, maps: int = 1,
+           merge=None) -> Optional[torch.Tensor]:
     """The step's tokens over the pages: tiles of query rows, key ranges split over blocks when the
     tiles are few.  In bfloat16 with keys and values of one width that the tcgen05 kernel takes,
     requests that bring more query rows than one tile of `ops.scaled_attention` holds go to it; the
     others, and all where it does not take the sizes, go to `ops.scaled_attention`: requests of few query
-    rows (decoded tokens) to its form for those, where there is one, the others to its form for many."""
+    rows (decoded tokens) to its form for those, where there is one, the others to its form for many.
+
+    `maps` > 1: a key row of `key_dim` columns is that many keys, `heads` counts the queries of all of
+    them.  With `merge` nothing is written to `out`: the kernels leave every key range's result, and
+    merge(part_o, part_ml, ranges, tokens (a list on the device, or None for all), their number) is
+    called behind each of them."""
     tokens = q.shape[0]
     # "mma": "auto" without the tcgen05 kernel (the entry point's own "mma" refuses what it cannot take)
     form = "auto" if FORM == "mma" else FORM
@@ -52,13 +59,15 @@ def attend(ctx, rt, q: torch.Tensor, head_scale: torch.Tensor, group, cache: Lay
     reach = min(window if window > 0 else chunk, chunk if chunk > 0 else window)   # 0: every key
 
     def scratch(nsplit: int):
-        if nsplit <= 1:
+        if nsplit <= 1 and merge is None:
             return None, None
         return (ctx.scratch("scaled_attention.part_o", nsplit * tokens * heads * value_dim),
                 ctx.scratch("scaled_attention.part_ml", nsplit * tokens * heads * 2))
 
+    extras = dict(chunk=chunk, softcap=softcap, gate=gate, head_gate=head_gate, sink=sink, pos_scale=pos_scale,
+                  maps=maps, partial=merge is not None)
     pages_map = None
-    if FORM == "auto" and form == "auto" and q.dtype is torch.bfloat16 and cache.pages is not None \
+    if FORM == "auto" and maps <= 2 and form == "auto" and q.dtype is torch.bfloat16 and cache.pages is not None \
             and (gate is None or (gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0)):
         pages_map = rt.pages_map(cache.pages)
     # (form, rows of its tiles) from few query rows to many; a request goes to the first whose tile
@@ -79,22 +88,27 @@ def attend(ctx, rt, q: torch.Tensor, head_scale: torch.Tensor, group, cache: Lay
             longest = min(longest, reach + class_rows)
         if class_form == "tcgen05":
             nsplit = attention_splits(tiles.count * kv_heads, longest, rt.sm_count, False, blocks_per_sm=1)
+            parts = scratch(nsplit)
             ops.attention_tc_scaled(pages_map, cache.entry_index, q, q.stride(0), head_scale,
                                     group.block_tables, tiles.item, tiles.row0, tiles.count,
                                     ctx.item_qstart, ctx.item_qlen, ctx.item_pos0, out, tokens, heads,
-                                    kv_heads, window, ctx.error, nsplit, *scratch(nsplit), chunk=chunk,
-                                    softcap=softcap, gate=gate, combine_tokens=class_tokens,
-                                    num_combine=count)
+                                    kv_heads, window, ctx.error, nsplit, *parts, combine_tokens=class_tokens,
+                                    num_combine=count, **extras)
+            if merge is not None:
+                merge(*parts, nsplit, class_tokens, count)
             continue
         nsplit = key_splits(tiles.count * kv_heads, longest, rt.sm_count,
                             key_tile=64 if q.dtype is torch.bfloat16 else 32)
+        parts = scratch(nsplit)
         ops.scaled_attention(q, q.stride(0), head_scale, cache.k_pages, cache.v_pages,
                              cache.page_stride, group.page_size, key_dim, value_dim,
                              values_in_keys, group.block_tables, tiles.item, tiles.row0,
                              tiles.count, ctx.item_qstart, ctx.item_qlen, ctx.item_pos0,
                              ctx.item_slots, out, tokens, heads, kv_heads, window, ctx.error,
-                             nsplit, *scratch(nsplit), form=class_form, chunk=chunk, softcap=softcap,
-                             gate=gate, combine_tokens=class_tokens, num_combine=count)
+                             nsplit, *parts, form=class_form, combine_tokens=class_tokens, num_combine=count,
+                             **extras)
+        if merge is not None:
+            merge(*parts, nsplit, class_tokens, count)
     return out
 
 
@@ -115,24 +129,29 @@ class ScaledGqaAttention(Mixer):
     from position 0 of the sequence (beside, or instead of, the window).  `qk_norm`: every head of q
     and of k is divided by its root mean square (`eps` inside the root) times a stored gain of `dim`
     numbers that all heads share, in 32-bit, before the rotation (`qk_gain`=False: no gain is stored,
-    the root mean square alone).  `head_gate`: every head's output is multiplied by
-    sigmoid(W_g y)[head], one number per head, before the output projection; `column_gate`: the
-    concatenated heads are multiplied element by element by sigmoid(W_g y), as the attention kernel
-    writes them.  W_g rides in the one product with q, k and v.
+    the root mean square alone; `norm_span` "projection": the root mean square is over all heads of q (of
+    k) at once, before they are split, and the gain is as wide).  `keys_as_values`: there is no v
+    projection, the values are the keys as projected, before norm and rotation.  `sink`: the
+    softmax's denominator also holds e^(stored number) per query head, which has no key, no value and no
+    scale.  `head_gate`: every head's output is multiplied by
+    sigmoid(W_g y)[head], one number per head; `column_gate`: the
+    concatenated heads are multiplied element by element by sigmoid(W_g y); both as the attention kernel
+    writes its result.  W_g rides in the one product with q, k and v.
     `names` gives the tensor names below the prefix.
     """
 
     capturable = True
 
     NAMES = {"q": "q", "k": "k", "v": "v", "o": "o", "bias": ".b", "temperature": "temp",
-             "mix": "vmix", "norm": ".norm", "gate": "g"}
+             "mix": "vmix", "norm": ".norm", "gate": "g", "sink": "sink"}
 
     def __init__(self, prefix: str, hidden_size: int, heads: int, kv_heads: int, dim: int,
                  vdim: int, scale: float, position: PartSpec, window: int = 0,
                  value_mix: str = "none", temperature: bool = True,
                  names: Optional[Dict[str, str]] = None, chunk: int = 0, qk_norm: bool = False,
                  eps: float = 0.0, head_gate: bool = False, bias: bool = True, softcap: float = 0.0,
-                 qk_gain: bool = True, column_gate: bool = False):
+                 qk_gain: bool = True, column_gate: bool = False, norm_span: str = "head",
+                 keys_as_values: bool = False, sink: bool = False):
         if heads % kv_heads:
             raise ValueError("heads must be a multiple of kv_heads")
         if value_mix not in ("none", "source", "mix"):
@@ -148,10 +167,16 @@ class ScaledGqaAttention(Mixer):
             raise ValueError("window, chunk and softcap must not be negative")
         if self.head_gate and self.column_gate:
             raise ValueError("scaled_gqa_attention: a gate per head or a gate per column, not both")
-        if (self.qk_norm or self.head_gate or self.column_gate) and value_mix != "none":
-            raise ValueError("scaled_gqa_attention: blended values go with neither qk_norm nor a gate")
+        self.keys_as_values, self.sink = bool(keys_as_values), bool(sink)
+        if norm_span not in ("head", "projection"):
+            raise ValueError("norm_span must be 'head' or 'projection'")
+        self.whole_norm = self.qk_norm and norm_span == "projection"
+        if (self.qk_norm or self.head_gate or self.column_gate or self.keys_as_values) and value_mix != "none":
+            raise ValueError("scaled_gqa_attention: blended values go with neither qk_norm nor a gate nor keys as values")
+        if self.keys_as_values and (self.vdim != self.dim or self.bias):
+            raise ValueError("scaled_gqa_attention: values that are the keys are as wide as they are, and have no bias")
         self.q_width, self.k_width = self.heads * self.dim, self.kv_heads * self.dim
-        self.v_width = self.kv_heads * self.vdim
+        self.v_width = 0 if self.keys_as_values else self.kv_heads * self.vdim      # columns of the projection
         self.gate_width = self.heads if self.head_gate else (self.heads * self.vdim if self.column_gate else 0)
         self.position = build_part("position", position, prefix)
         if self.position.rotary_dim > self.dim:
@@ -161,12 +186,15 @@ class ScaledGqaAttention(Mixer):
         self.names = dict(self.NAMES)
         self.names.update(names or {})
         self.w_qkv = self.b_qkv = self.w_o = self.head_scale = self.mix = None
-        self.q_gain = self.k_gain = None
+        self.q_gain = self.k_gain = self.sinks = None
+
+    def _projections(self):
+        return "qk" if self.keys_as_values else "qkv"
 
     def tensor_specs(self) -> List[TensorSpec]:
         p, h, n = self.prefix, self.hidden_size, self.names
         specs = []
-        for which, width in (("q", self.q_width), ("k", self.k_width), ("v", self.v_width)):
+        for which, width in zip(self._projections(), (self.q_width, self.k_width, self.v_width)):
             specs.append(TensorSpec(p + n[which], (width, h)))
             if self.bias:
                 specs.append(TensorSpec(p + n[which] + n["bias"], (width,)))
@@ -175,8 +203,10 @@ class ScaledGqaAttention(Mixer):
         if self.temperature:
             specs.append(TensorSpec(p + n["temperature"], (self.heads,), role="vector", init="gain"))
         if self.qk_norm and self.qk_gain:
-            specs += [TensorSpec(p + n[which] + n["norm"], (self.dim,), role="vector", init="gain")
-                      for which in ("q", "k")]
+            specs += [TensorSpec(p + n[which] + n["norm"], (width if self.whole_norm else self.dim,), role="vector",
+                                 init="gain") for which, width in (("q", self.q_width), ("k", self.k_width))]
+        if self.sink:
+            specs.append(TensorSpec(p + n["sink"], (self.heads,), role="vector", init="normal"))
         if self.gate_width:
             specs.append(TensorSpec(p + n["gate"], (self.gate_width, h)))
         specs.append(TensorSpec(p + n["o"], (h, self.heads * self.vdim)))
@@ -193,7 +223,7 @@ class ScaledGqaAttention(Mixer):
     def bind(self, tensors: Dict[str, torch.Tensor], runtime) -> None:
         self.runtime = runtime
         p, n = self.prefix, self.names
-        stacked = [tensors[p + n[k]] for k in "qkv"]
+        stacked = [tensors[p + n[k]] for k in self._projections()]
         if self.gate_width:                 # the gate's rows behind q, k and v; it has no bias
             stacked.append(tensors[p + n["gate"]])
         rows = sum(w.shape[0] for w in stacked)
@@ -210,6 +240,8 @@ class ScaledGqaAttention(Mixer):
         if self.qk_norm and self.qk_gain:
             self.q_gain = tensors[p + n["q"] + n["norm"]].to(torch.float32).contiguous()
             self.k_gain = tensors[p + n["k"] + n["norm"]].to(torch.float32).contiguous()
+        if self.sink:
+            self.sinks = tensors[p + n["sink"]].to(torch.float32).contiguous()
         self.w_o = tensors[p + n["o"]].contiguous()
         scale = torch.full((self.heads,), self.scale, dtype=torch.float32, device=runtime.device)
         if self.temperature:
@@ -237,11 +269,12 @@ class ScaledGqaAttention(Mixer):
             if v_first is None or v_first.shape != (tokens, self.v_width):
                 raise ValueError("scaled_gqa_attention: no layer before this one has left values "
                                  "of this width to blend with")
-        if self.qk_norm or self.gate_width:
+        if self.qk_norm or self.gate_width or self.keys_as_values:
             ops.norm_rotate_write(qkv, ctx.positions, self.position.table, group.slot_of, cache.k_pages,
                                   cache.v_pages, cache.page_stride, group.page_size, self.heads,
                                   self.kv_heads, self.dim, self.vdim, self.position.rotary_dim,
-                                  self.q_gain, self.k_gain, self.eps, ctx.error, unit=self.qk_norm)
+                                  self.q_gain, self.k_gain, self.eps, ctx.error, unit=self.qk_norm,
+                                  whole=self.whole_norm, values_from_keys=self.keys_as_values)
         else:
             ops.rotate_mix_write(qkv, ctx.positions, self.position.table, group.slot_of, cache.k_pages,
                                  cache.v_pages, cache.page_stride, group.page_size, self.heads,
@@ -251,7 +284,6 @@ class ScaledGqaAttention(Mixer):
         gate0 = self.q_width + self.k_width + self.v_width
         gate = qkv[:, gate0:gate0 + self.gate_width] if self.gate_width else None
         attend(ctx, rt, qkv, self.head_scale, group, cache, out, self.heads, self.kv_heads, self.dim,
-               self.vdim, False, self.window, self.chunk, self.softcap, gate if self.column_gate else None)
-        if self.head_gate:
-            ops.head_gate(out, gate, self.heads, self.vdim)
+               self.vdim, False, self.window, self.chunk, self.softcap, gate if self.column_gate else None,
+               gate if self.head_gate else None, self.sinks)
         return rt.linear(out, self.w_o, None, "scaled_attention.o")

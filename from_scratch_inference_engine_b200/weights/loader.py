@@ -35,8 +35,9 @@ def check_tensors(specs: Iterable[TensorSpec], tensors: Mapping[str, torch.Tenso
     unexpected = [name for name in tensors if name not in declared]
     wrong = []
     for name, spec in declared.items():
-        if name in tensors and tuple(tensors[name].shape) != tuple(spec.shape):
-            wrong.append(f"{name}: expected {list(spec.shape)}, found "
+        if name in tensors and not spec.fits(tensors[name].shape):
+            expected = [f"any ({size})" if axis in spec.free else size for axis, size in enumerate(spec.shape)]
+            wrong.append(f"{name}: expected [{', '.join(map(str, expected))}], found "
                          f"{list(tensors[name].shape)}")
     unequal = []
     for name, spec in declared.items():

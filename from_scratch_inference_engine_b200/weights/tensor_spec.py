@@ -3,7 +3,7 @@
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Tuple
+from typing import Sequence, Tuple
 
 
 @dataclass(frozen=True)
@@ -19,6 +19,8 @@ class TensorSpec:
               weight) or "eye" (identity + N(0, std):
               a matrix that mixes heads).
     optional  may be absent from the checkpoint (the part says what it does then).
+    free      dimensions whose size the checkpoint decides (a size that no configuration key gives);
+              `shape` then holds what the random-weights mode draws.
     same_as   when present in the checkpoint it must equal this other tensor
               (a head tied to the embedding that is stored a second time).
     """
@@ -29,3 +31,10 @@ class TensorSpec:
     init: str = "normal"
     optional: bool = False
     same_as: str = ""
+    free: Tuple[int, ...] = ()
+
+    def fits(self, shape: Sequence[int]) -> bool:
+        """Whether a stored tensor of `shape` is one of this kind."""
+        return len(shape) == len(self.shape) and all(
+            have == want or (axis in self.free and have > 0)
+            for axis, (have, want) in enumerate(zip(shape, self.shape)))

@@ -148,19 +148,6 @@ def test_heads_normed_then_turned_into_the_cache(dtype, normed):
     assert float(kp.abs().sum(dim=(1, 3)).ne(0).sum()) == 8          # one token had no slot: nothing stored
 
 
-@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-def test_gate_per_head(dtype):
-    from from_scratch_inference_engine_b200.kernels import ops
-    g = torch.Generator().manual_seed(4)
-    for heads, vdim in ((3, 10), (8, 64)):
-        out = torch.randn(11, heads * vdim, generator=g).to(dtype)
-        wide = torch.randn(11, heads + 9, generator=g).to(dtype).cuda()
-        got = ops.head_gate(out.clone().cuda(), wide[:, 5:5 + heads], heads, vdim)
-        want = out.double().view(11, heads, vdim) * torch.sigmoid(wide[:, 5:5 + heads].cpu().double())[:, :, None]
-        tolerance = 1e-6 if dtype is torch.float32 else 2e-2
-        assert (got.cpu().double().view(11, heads, vdim) - want).abs().max() < tolerance * 4
-
-
 def _paged(rows, page_size, order, pages_total):
     """rows [n, kv_heads, width] laid out as pages [kv_head][slot][width] at the given page ids."""
     n, kv_heads, width = rows.shape

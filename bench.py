@@ -29,7 +29,9 @@ Kufulix design (windowed attention beside a state-space mixer, chunked attention
 without gates) beside a Metulix model of equal size; `--workload deginex` measures the Deginex design (a
 residual of four streams, chunked attention with unit q and k, capped scores and a gate per column, dense
 and routed feed-forwards in turn, a looped stretch) beside a Kufulix model of chunked attention layers of
-equal size; `--workload tapalix` measures the
+equal size; `--workload lanilorn` measures the Lanilorn design (a residual of four streams; differential
+attention, windowed attention with sinks whose values are its keys, gated linear attention; feed-forwards of
+squared relu) beside a Deginex model of as many streams and heads; `--workload tapalix` measures the
 Tapalix design (latent attention with and without a rotated part, routed experts beside a shared one,
 a looped stretch of layers) beside a Zadepel model of latent attention layers with a dense feed-forward
 of the width a token uses, at equal depth.
@@ -559,6 +561,38 @@ def deginex_shapes(width, heads, kv_heads, dim, streams, dense, experts, top, ff
     return deginex, kufulix
 
 
+# name, width, heads, kv heads, head size, streams, feed-forward, recurrent heads, their key and value sizes,
+# layers, vocabulary
+LANILORN_SIZES = (("w2048", 2048, 16, 4, 128, 4, 9216, 16, 64, 128, 4, 32000),
+                  ("w4096", 4096, 32, 8, 128, 4, 18432, 32, 64, 128, 4, 32000))
+
+
+def lanilorn_shapes(width, heads, kv_heads, dim, streams, ff, gla_heads, gla_dim, gla_vdim, layers, vocab, window):
+    """A Lanilorn model (differential, windowed, recurrent and windowed layers in turn, the recurrent ones without
+    a feed-forward) and the closest model the engine had: a Deginex model of as many streams and heads, full
+    causal attention where the other is differential or recurrent, chunks of two windows (as many keys on
+    average) where it is windowed, its gated feed-forward two thirds as wide so that the matrices hold as many
+    numbers."""
+    kinds = ("attention_2", "attention", "gla", "attention")
+    heads_of = {"heads": heads, "kv_heads": kv_heads, "vdim": dim, "scale": dim ** -0.5}
+    mixers = {"attention": dict(heads_of, dim=dim, mask={"size": window}, rot={
+                  "base": 250000.0, "dims": dim // 2,
+                  "scaling": {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}}),
+              "attention_2": dict(heads_of, dim=dim // 2, diff=0.6, q_temp={"coef": 0.3, "every": 64}),
+              "gla": {"heads": gla_heads, "dim": gla_dim, "vdim": gla_vdim, "tau": 16.0}}
+    order = [kinds[i % len(kinds)] for i in range(layers)]
+    lanilorn = {"architecture": "Lanilorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+                "streams": streams, "embedding": {"scale": 0.5}, "logit_scale": 0.25,
+                "layers": [{"type": kind, "mixer": mixers[kind],
+                            "mlp": None if kind == "gla" else {"kind": "dense", "ff": ff}} for kind in order]}
+    beside = {"attention": dict(heads_of, dim=dim, mask={"size": 2 * window}), "full": dict(heads_of, dim=dim)}
+    deginex = {"architecture": "Deginex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+               "streams": streams, "loop": None,
+               "layers": [{"type": "attention", "mixer": beside.get(kind, beside["full"]),
+                           "mlp": None if kind == "gla" else {"kind": "dense", "ff": ff * 2 // 3}} for kind in order]}
+    return lanilorn, deginex
+
+
 def hybrid_workload(args, design="metulix") -> int:
     """The Metulix design (or, `design`, the Zadepel design) beside the Qwen2 model of equal size
     (random bf16 weights): prefill of
@@ -596,8 +630,9 @@ def hybrid_workload(args, design="metulix") -> int:
                                "scaled_attention", "rotate_mix_write", "latent_prep", "head_product",
                                "sum_layernorm", "settle_concat", "logit_cap", "sigmoid_gate", "moe_route",
                                "moe_align", "moe_gather", "moe_product", "gemm_tiles_grouped", "moe_combine",
-                               "ssd_prep", "ssd_tails", "ssd_gate_norm", "norm_rotate_write", "head_gate",
-                               "scaled_sum_rmsnorm", "stream_norm", "attention_tc_scaled")
+                               "ssd_prep", "ssd_tails", "ssd_gate_norm", "norm_rotate_write",
+                               "scaled_sum_rmsnorm", "stream_norm", "attention_tc_scaled", "difference_merge",
+                               "row_decay", "head_norm_silu", "relu_squared")
              if hasattr(ops, name)]
 
     def by_kind(fn):
@@ -633,7 +668,8 @@ def hybrid_workload(args, design="metulix") -> int:
         out["(whole step)"] = total
         return {k: round(v, 4) for k, v in sorted(out.items(), key=lambda kv: -kv[1])}
 
-    table = {"tapalix": TAPALIX_SIZES, "kufulix": KUFULIX_SIZES, "deginex": DEGINEX_SIZES}.get(design, HYBRID_SIZES)
+    table = {"tapalix": TAPALIX_SIZES, "kufulix": KUFULIX_SIZES, "deginex": DEGINEX_SIZES,
+             "lanilorn": LANILORN_SIZES}.get(design, HYBRID_SIZES)
     sizes = [s for s in table if not args.sizes or s[0] in args.sizes.split(",")]
     results = []
     clocks = ClockSampler()
@@ -670,6 +706,15 @@ def hybrid_workload(args, design="metulix") -> int:
                      "layers": layers, "passes": times, "layer_runs": len(shapes[1]["layers"]), "vocab": vocab,
                      "chunk": 2 * window}
             beside = "kufulix"
+        elif design == "lanilorn":
+            (name, width, heads, kv_heads, dim, streams, ff, gla_heads, gla_dim, gla_vdim, layers, vocab) = size
+            layers = args.layers or layers
+            shapes = lanilorn_shapes(width, heads, kv_heads, dim, streams, ff, gla_heads, gla_dim, gla_vdim,
+                                     layers, vocab, window)
+            entry = {"size": name, "width": width, "heads": heads, "kv_heads": kv_heads, "head_dim": dim,
+                     "streams": streams, "ff": ff, "gla": {"heads": gla_heads, "dim": gla_dim, "vdim": gla_vdim},
+                     "layers": layers, "vocab": vocab, "window": window}
+            beside = "deginex"
         else:
             name, width, heads, kv_heads, dim, ff, layers, vocab = size
             layers = args.layers or layers
@@ -745,7 +790,7 @@ def hybrid_workload(args, design="metulix") -> int:
     clock_record = clocks.stop()
     print(json.dumps({
         "metric": f"prefill and decode tokens/s of the {design.capitalize()} design beside "
-                  f"{ {'tapalix': 'Zadepel', 'kufulix': 'Metulix', 'deginex': 'Kufulix'}.get(design, 'Qwen2') } at equal size",
+                  f"{ {'tapalix': 'Zadepel', 'kufulix': 'Metulix', 'deginex': 'Kufulix', 'lanilorn': 'Deginex'}.get(design, 'Qwen2') } at equal size",
         "impl": "engine", "unit": "tokens/s", "n_gpus": 1, "steps": steps, "warmup": warmup,
         "dtype": "bf16" if compute == "bfloat16" else "fp32",
         "config": {"prefill_tokens": prompt_len, "decode_batch": batch, "decode_context": context,
@@ -836,7 +881,7 @@ def main() -> int:
     parser.add_argument("--fp32-steps", type=int, default=8,
                         help="decode steps timed on the float32 path after the bf16 run (0 = skip)")
     parser.add_argument("--workload", default="decode", choices=["decode", "serving", "long", "timeline", "hybrid", "zadepel", "tapalix", "kufulix",
-                                                                        "deginex"],
+                                                                        "deginex", "lanilorn"],
                         help="decode: the default measurement; serving: continuous batching of 256 "
                              "requests at the 1.5B shape; long: the 14B shape, decode at batch 32 with "
                              "8,192-token contexts and chunked prefill of an 8,192-token prompt; "
@@ -845,6 +890,7 @@ def main() -> int:
                              "zadepel: the same for the Zadepel design; "
                              "kufulix: the Kufulix design beside a Metulix model; "
                              "deginex: the Deginex design beside a Kufulix model of chunked attention layers; "
+                             "lanilorn: the Lanilorn design beside a Deginex model of as many streams and heads; "
                              "tapalix: the Tapalix design beside a Zadepel model of latent attention layers")
     parser.add_argument("--sizes", default="", help="hybrid: which sizes to run (w2048,w4096; '' = all)")
     parser.add_argument("--requests", type=int, default=256)
@@ -877,6 +923,8 @@ def main() -> int:
         return hybrid_workload(args, design="kufulix")
     if args.workload == "deginex":
         return hybrid_workload(args, design="deginex")
+    if args.workload == "lanilorn":
+        return hybrid_workload(args, design="lanilorn")
 
     import numpy as np
     import torch

@@ -34,6 +34,11 @@ __device__ __forceinline__ float4 scan_load4(const bf16* p) {
     const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
     return make_float4(a.x, a.y, b.x, b.y);
 }
+__device__ __forceinline__ void scan_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void scan_store4(bf16* p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
 
 // where row d of a staged q or k vector lives: the DR rows of a thread are contiguous (one or
 // more 16-byte loads) and the groups are four floats apart in the banks
@@ -183,23 +188,18 @@ lightning_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, 
                     if (write_out) o[x] += s[i][x] * qq[i];
                 }
             if (!write_out) continue;
-#pragma unroll
-            for (int x = 0; x < 4; ++x) {
-                o[x] += __shfl_xor_sync(0xffffffffu, o[x], 1);
-                o[x] += __shfl_xor_sync(0xffffffffu, o[x], 2);
-                o[x] += __shfl_xor_sync(0xffffffffu, o[x], 4);
-                o[x] += __shfl_xor_sync(0xffffffffu, o[x], 8);
-            }
-            if (rg == 0 && col0 < vdim) {
-#pragma unroll
-                for (int x = 0; x < 4; ++x) o[x] *= out_scale;
-                float* dst = out + (size_t)(start + t0 + t) * heads * vdim + head * vdim + col0;
-                if (wide) *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]);
-                else {
-#pragma unroll
-                    for (int x = 0; x < 4; ++x) if (col0 + x < vdim) dst[x] = o[x];
-                }
-            }
+            // the sum over the 16 row groups: the first two exchanges halve what a lane holds (four columns,
+            // two, one), the last two add one column's parts; five exchanges, not sixteen
+            const bool upper = rg & 1, odd = rg & 2;
+            const float a0 = __shfl_xor_sync(0xffffffffu, upper ? o[0] : o[2], 1);
+            const float a1 = __shfl_xor_sync(0xffffffffu, upper ? o[1] : o[3], 1);
+            const float b0 = (upper ? o[2] : o[0]) + a0, b1 = (upper ? o[3] : o[1]) + a1;
+            float sum = (odd ? b1 : b0) + __shfl_xor_sync(0xffffffffu, odd ? b0 : b1, 2);
+            sum += __shfl_xor_sync(0xffffffffu, sum, 4);
+            sum += __shfl_xor_sync(0xffffffffu, sum, 8);
+            const int col = col0 + (upper ? 2 : 0) + (odd ? 1 : 0);
+            if (rg < 4 && col < vdim)
+                out[(size_t)(start + t0 + t) * heads * vdim + head * vdim + col] = sum * out_scale;
         }
     }
     if (!ROWS && phase == 1 && chunk_decay && blockIdx.x == 0 && threadIdx.x == 0)
@@ -328,7 +328,8 @@ __global__ void row_decay_kernel(const T* __restrict__ proj, int ld, int low_off
 
 // A warp per (token, head): y = T( o / sqrt(mean(o^2) + eps) * gain * silu(gate) ), the mean over the head's vdim
 // columns, the gain [vdim] shared by the heads.
-template <typename T>
+// VEC columns side by side per lane.
+template <typename T, int VEC>
 __global__ void head_norm_silu_kernel(const float* __restrict__ o, const T* __restrict__ proj, int ld, int g_off,
                                       const float* __restrict__ gain, T* __restrict__ y, long long pairs, int heads,
                                       int vdim, float eps) {
@@ -343,9 +344,24 @@ __global__ void head_norm_silu_kernel(const float* __restrict__ o, const T* __re
     const T* gate = proj + t * ld + g_off + (size_t)h * vdim;
     T* yr = y + pair * vdim;
     float sq = 0.f;
-    for (int c = lane; c < vdim; c += 32) sq += row[c] * row[c];
+    for (int c = lane * VEC; c < vdim; c += 32 * VEC) {
+        if (VEC == 4) {
+            const float4 v = scan_load4(row + c);
+            sq += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+        } else {
+            sq += row[c] * row[c];
+        }
+    }
     const float inv = 1.0f / sqrtf(warp_sum(sq) / (float)vdim + eps);
-    for (int c = lane; c < vdim; c += 32) yr[c] = from_float<T>(row[c] * inv * gain[c] * silu_f(to_float(gate[c])));
+    for (int c = lane * VEC; c < vdim; c += 32 * VEC) {
+        if (VEC == 4) {
+            const float4 v = scan_load4(row + c), w = scan_load4(gain + c), z = scan_load4(gate + c);
+            scan_store4(yr + c, make_float4(v.x * inv * w.x * silu_f(z.x), v.y * inv * w.y * silu_f(z.y),
+                                            v.z * inv * w.z * silu_f(z.z), v.w * inv * w.w * silu_f(z.w)));
+        } else {
+            yr[c] = from_float<T>(row[c] * inv * gain[c] * silu_f(to_float(gate[c])));
+        }
+    }
 }
 
 // One block per token: y = T( o * rsqrt(mean(o^2) + eps) * gain * sigmoid(gate) ).
@@ -480,11 +496,13 @@ int fsie_head_norm_silu(const float* o, const void* proj, int ld, int g_off, con
     const long long pairs = (long long)tokens * heads;
     if (pairs <= 0 || vdim <= 0) return 0;
     const dim3 grid((unsigned)((pairs + 3) / 4));
-    if (dtype == DTYPE_F32)
-        return launch_dependent(head_norm_silu_kernel<float>, grid, dim3(128), 0, stream, o, (const float*)proj, ld, g_off,
-                                gain, (float*)y, pairs, heads, vdim, eps);
-    return launch_dependent(head_norm_silu_kernel<bf16>, grid, dim3(128), 0, stream, o, (const bf16*)proj, ld, g_off, gain,
-                            (bf16*)y, pairs, heads, vdim, eps);
+    const bool vec = ((vdim | ld | g_off) & 3) == 0 && (((size_t)o | (size_t)gain | (size_t)proj | (size_t)y) & 15) == 0;
+#define FSIE_HEAD_NORM(T, V)                                                                                     \
+    launch_dependent(head_norm_silu_kernel<T, V>, grid, dim3(128), 0, stream, o, (const T*)proj, ld, g_off, gain, \
+                     (T*)y, pairs, heads, vdim, eps)
+    if (dtype == DTYPE_F32) return vec ? FSIE_HEAD_NORM(float, 4) : FSIE_HEAD_NORM(float, 1);
+    return vec ? FSIE_HEAD_NORM(bf16, 4) : FSIE_HEAD_NORM(bf16, 1);
+#undef FSIE_HEAD_NORM
 }
 
 int fsie_gated_rmsnorm(const float* o, const void* proj, int ld, int g_off, const float* gain,

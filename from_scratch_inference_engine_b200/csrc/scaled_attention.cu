@@ -1125,9 +1125,7 @@ __global__ void rotate_mix_write_kernel(T* __restrict__ proj, int ld, const int*
 //          then pairs (i, i + rotary_dim / 2) turn by the token's angles; q in place, k into its page
 //   v      into its page as it is; with `v_from_k` the projection holds no v, and the values are the
 //          keys as they were projected (vdim = dim)
-// VEC: head sizes are multiples of 8 and every row and page starts on 16 bytes: eight
-// columns per lane and trip.
-template <typename T, bool VEC>
+template <typename T>
 __global__ void norm_rotate_write_kernel(T* __restrict__ proj, int ld, const int* __restrict__ positions,
                                          const float* __restrict__ cos_sin, int table_len,
                                          const int* __restrict__ slot_of, T* __restrict__ k_pages,
@@ -1137,7 +1135,6 @@ __global__ void norm_rotate_write_kernel(T* __restrict__ proj, int ld, const int
                                          float eps, int unit, int whole, int v_from_k, int* __restrict__ error) {
     extern __shared__ __align__(32) float nr_smem[];   // [warps][dim]
     __shared__ float scratch[32];
-    constexpr int STEP = VEC ? 8 : 1;
     const int t = blockIdx.x;
     grid_dependency_wait();
     grid_dependents_go();
@@ -1161,12 +1158,9 @@ __global__ void norm_rotate_write_kernel(T* __restrict__ proj, int ld, const int
             const T* src = row + (side ? (size_t)heads * dim : 0);
             const int columns = (side ? kv_heads : heads) * dim;
             float sq = 0.f;
-            for (int d = threadIdx.x * STEP; d < columns; d += blockDim.x * STEP) {
-                float v[8];
-                if (VEC) load8(src + d, v);
-                else v[0] = to_float(src[d]);
-#pragma unroll
-                for (int i = 0; i < STEP; ++i) sq += v[i] * v[i];
+            for (int d = threadIdx.x; d < columns; d += blockDim.x) {
+                const float v = to_float(src[d]);
+                sq += v * v;
             }
             whole_inv[side] = 1.0f / sqrtf(block_sum(sq, scratch) / (float)columns + eps);
         }
@@ -1178,54 +1172,139 @@ __global__ void norm_rotate_write_kernel(T* __restrict__ proj, int ld, const int
         const float* gain = is_q ? q_gain : k_gain;
         if (whole && gain) gain += (size_t)(is_q ? h : h - heads) * dim;
         float sq = 0.f;
-        for (int d = lane * STEP; d < dim; d += 32 * STEP) {
-            float v[8];
-            if (VEC) load8(src + d, v);
-            else v[0] = to_float(src[d]);
-#pragma unroll
-            for (int i = 0; i < STEP; ++i) sq += v[i] * v[i];
-            if (VEC) store8(mine + d, v);
-            else mine[d] = v[0];
+        for (int d = lane; d < dim; d += 32) {
+            const float v = to_float(src[d]);
+            sq += v * v;
+            mine[d] = v;
         }
         if (gain || unit) {
             const float inv = whole ? whole_inv[is_q ? 0 : 1] : 1.0f / sqrtf(warp_sum(sq) / (float)dim + eps);
             // every lane changes what it wrote itself
-            for (int d = lane * STEP; d < dim; d += 32 * STEP)
-#pragma unroll
-                for (int i = 0; i < STEP; ++i) mine[d + i] = gain ? mine[d + i] * inv * gain[d + i] : mine[d + i] * inv;
+            for (int d = lane; d < dim; d += 32) mine[d] = gain ? mine[d] * inv * gain[d] : mine[d] * inv;
         }
         __syncwarp();
         T* dst = is_q ? src : k_pages + page * page_stride + ((long long)(h - heads) * page_size + off) * dim;
-        for (int d0 = lane * STEP; d0 < dim; d0 += 32 * STEP) {
-            float val[8];
-#pragma unroll
-            for (int j = 0; j < STEP; ++j) {
-                const int d = d0 + j;
-                val[j] = mine[d];
-                if (d < rotary_dim) {
-                    const int i = d < half ? d : d - half;
-                    const float c = cs[i], sn = cs[half + i];
-                    const float other = mine[d < half ? d + half : d - half];
-                    val[j] = d < half ? val[j] * c - other * sn : val[j] * c + other * sn;
-                }
+        for (int d = lane; d < dim; d += 32) {
+            float val = mine[d];
+            if (d < rotary_dim) {
+                const int i = d < half ? d : d - half;
+                const float c = cs[i], sn = cs[half + i];
+                const float other = mine[d < half ? d + half : d - half];
+                val = d < half ? val * c - other * sn : val * c + other * sn;
             }
-            if (VEC) store8(dst + d0, val);
-            else dst[d0] = from_float<T>(val[0]);
+            dst[d] = from_float<T>(val);
         }
         __syncwarp();
     }
     if (slot < 0) return;
     const T* v = row + (size_t)(v_from_k ? heads : heads + kv_heads) * dim;
-    for (int e = threadIdx.x * STEP; e < kv_heads * vdim; e += blockDim.x * STEP) {
+    for (int e = threadIdx.x; e < kv_heads * vdim; e += blockDim.x) {
         const int g = e / vdim, d = e - g * vdim;
-        T* dst = v_pages + page * page_stride + ((long long)g * page_size + off) * vdim + d;
-        if (VEC) {
-            float val[8];
-            load8(v + e, val);
-            store8(dst, val);
-        } else {
-            *dst = v[e];
+        v_pages[page * page_stride + ((long long)g * page_size + off) * vdim + d] = v[e];
+    }
+}
+
+// The same where rows and pages start on 16 bytes, head sizes are multiples of 8 and the rotated width of 16:
+// a thread holds NCH chunks of eight columns of the token's row in registers - one trip to memory, every
+// chunk written once.  Root mean squares are added up and rotation partners met through shared memory.
+// Chunks are q's, then k's, then v's (where the projection has any); q is left out where nothing changes it.
+template <typename T, int NCH>
+__global__ void __launch_bounds__(512) norm_rotate_rows_kernel(
+        T* __restrict__ proj, int ld, const int* __restrict__ positions, const float* __restrict__ cos_sin, int table_len,
+        const int* __restrict__ slot_of, T* __restrict__ k_pages, T* __restrict__ v_pages, long long page_stride,
+        int page_size, int heads, int kv_heads, int dim, int vdim, int rotary_dim, const float* __restrict__ q_gain,
+        const float* __restrict__ k_gain, float eps, int unit, int whole, int v_from_k, int first_chunk,
+        int* __restrict__ error) {
+    extern __shared__ __align__(32) float nr_smem[];   // [chunks of q and k] sums of squares, then their columns
+    __shared__ float scratch[32];
+    const int t = blockIdx.x;
+    const int per_head = dim / 8, chunks_q = heads * per_head, chunks_qk = chunks_q + kv_heads * per_head;
+    const int chunks = chunks_qk + (v_from_k ? 0 : kv_heads * vdim / 8);
+    float* part = nr_smem;
+    float* columns = nr_smem + (chunks_qk + 7) / 8 * 8;
+    // where the token sits was staged before the step
+    const int pos = positions[t];
+    const int slot = slot_of ? slot_of[t] : -1;
+    grid_dependency_wait();
+    grid_dependents_go();
+    if (rotary_dim > 0 && (pos < 0 || pos >= table_len)) {
+        if (threadIdx.x == 0) atomicExch(error, 2);
+        return;
+    }
+    const int half = rotary_dim / 2;
+    const float* cs = cos_sin + (size_t)pos * rotary_dim;
+    T* row = proj + (size_t)t * ld;
+    const long long page = slot >= 0 ? slot / page_size : -1;
+    const int off = slot >= 0 ? slot % page_size : 0;
+    float v[NCH][8], sq_q = 0.f, sq_k = 0.f;
+#pragma unroll
+    for (int i = 0; i < NCH; ++i) {
+        const int c = first_chunk + threadIdx.x + i * blockDim.x;
+        if (c < chunks) load8(row + (size_t)c * 8, v[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < NCH; ++i) {
+        const int c = first_chunk + threadIdx.x + i * blockDim.x;
+        if (c >= chunks) continue;
+        if (slot >= 0 && c >= (v_from_k ? chunks_q : chunks_qk)) {          // a value, as it is
+            const int e = (c - (v_from_k ? chunks_q : chunks_qk)) * 8;
+            const int g = e / vdim;
+            store8(v_pages + page * page_stride + ((long long)g * page_size + off) * vdim + (e - g * vdim), v[i]);
         }
+        if (c >= chunks_qk) continue;
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) s += v[i][j] * v[i][j];
+        if (c < chunks_q) sq_q += s;
+        else sq_k += s;
+        if (!whole) part[c] = s;
+    }
+    const bool norm_q = q_gain || unit, norm_k = k_gain || unit;
+    float inv_q = 1.f, inv_k = 1.f;
+    if (whole) {
+        inv_q = 1.0f / sqrtf(block_sum(sq_q, scratch) / (float)(heads * dim) + eps);
+        inv_k = 1.0f / sqrtf(block_sum(sq_k, scratch) / (float)(kv_heads * dim) + eps);
+    } else if (norm_q || norm_k) {
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < NCH; ++i) {
+        const int c = first_chunk + threadIdx.x + i * blockDim.x;
+        if (c >= chunks_qk) continue;
+        const bool is_q = c < chunks_q;
+        const int h = c / per_head, d = (c - h * per_head) * 8;
+        if (is_q ? norm_q : norm_k) {
+            float inv = is_q ? inv_q : inv_k;
+            if (!whole) {
+                float s = 0.f;
+                for (int j = 0; j < per_head; ++j) s += part[h * per_head + j];
+                inv = 1.0f / sqrtf(s / (float)dim + eps);
+            }
+            const float* gain = is_q ? q_gain : k_gain;
+            float w[8];
+            if (gain) load8(gain + (whole ? (is_q ? h : h - heads) * dim : 0) + d, w);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[i][j] = gain ? v[i][j] * inv * w[j] : v[i][j] * inv;
+        }
+        if (d < rotary_dim) store8(columns + (size_t)c * 8, v[i]);
+    }
+    if (rotary_dim > 0) __syncthreads();
+#pragma unroll
+    for (int i = 0; i < NCH; ++i) {
+        const int c = first_chunk + threadIdx.x + i * blockDim.x;
+        if (c >= chunks_qk) continue;
+        const int h = c / per_head, d = (c - h * per_head) * 8;
+        if (d < rotary_dim) {                       // a chunk lies on one side of the rotation: half is a multiple of 8
+            const bool low = d < half;
+            float other[8], co[8], sn[8];
+            load8(columns + (size_t)c * 8 + (low ? half : -half), other);
+            load8(cs + (low ? d : d - half), co);
+            load8(cs + half + (low ? d : d - half), sn);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[i][j] = low ? v[i][j] * co[j] - other[j] * sn[j] : v[i][j] * co[j] + other[j] * sn[j];
+        }
+        if (c < chunks_q) store8(row + (size_t)c * 8, v[i]);
+        else if (slot >= 0) store8(k_pages + page * page_stride + ((long long)(h - heads) * page_size + off) * dim + d, v[i]);
     }
 }
 
@@ -1479,21 +1558,34 @@ int fsie_norm_rotate_write(void* proj, int ld, const int* positions, const float
     if (rotary_dim < 0 || rotary_dim > dim || (rotary_dim & 1) || dim <= 0 || (v_from_k && vdim != dim) ||
         ld < (heads + kv_heads) * dim + (v_from_k ? 0 : kv_heads * vdim))
         return ERR_BAD_ARGUMENT;
+    const size_t bits = (size_t)proj | (size_t)k_pages | (size_t)v_pages | (size_t)q_gain | (size_t)k_gain | (size_t)cos_sin;
+    const int columns = (heads + kv_heads) * dim;
+    const int first = (unit || q_gain || rotary_dim > 0) ? 0 : heads * dim / 8;      // nothing changes q: left where it is
+    const int chunks = columns / 8 + (v_from_k ? 0 : kv_heads * vdim / 8) - first;
+    const int each = (chunks + 511) / 512;
+    const size_t rows_smem = ((size_t)(columns / 8 + 7) / 8 * 8 + columns) * sizeof(float);
+    if (dim % 8 == 0 && vdim % 8 == 0 && rotary_dim % 16 == 0 && ld % 8 == 0 && page_stride % 8 == 0 && (bits & 15) == 0 &&
+        each <= 4 && rows_smem <= 48 * 1024) {
+        const int threads = ((chunks + each - 1) / each + 31) / 32 * 32;
+#define FSIE_NORM_ROWS(T, N)                                                                                        \
+    launch_dependent(norm_rotate_rows_kernel<T, N>, dim3(tokens), dim3(threads), rows_smem, stream, (T*)proj, ld,   \
+                     positions, cos_sin, table_len, slot_of, (T*)k_pages, (T*)v_pages, page_stride, page_size,     \
+                     heads, kv_heads, dim, vdim, rotary_dim, q_gain, k_gain, eps, unit, whole, v_from_k, first, error)
+#define FSIE_NORM_ROWS_SIZE(T) \
+    (each == 1 ? FSIE_NORM_ROWS(T, 1) : each == 2 ? FSIE_NORM_ROWS(T, 2) : each == 3 ? FSIE_NORM_ROWS(T, 3) : FSIE_NORM_ROWS(T, 4))
+        return dtype == DTYPE_F32 ? FSIE_NORM_ROWS_SIZE(float) : FSIE_NORM_ROWS_SIZE(bf16);
+#undef FSIE_NORM_ROWS_SIZE
+#undef FSIE_NORM_ROWS
+    }
     // a token's heads share a block; where tokens are few, a warp for each head
     const int warps = tokens <= 64 ? (heads + kv_heads < 16 ? heads + kv_heads : 16) : 8;
     const size_t smem = (size_t)warps * dim * sizeof(float);
     if (smem > 48 * 1024) return ERR_UNSUPPORTED;
-    const size_t bits = (size_t)proj | (size_t)k_pages | (size_t)v_pages;
-    // one trip to memory per head matters where tokens are few; with many, a column per lane measured
-    // faster (2,048 tokens x 20 heads of 128: 20 against 26 us)
-    const bool vec = tokens <= 64 && dim % 8 == 0 && vdim % 8 == 0 && ld % 8 == 0 && page_stride % 8 == 0 &&
-                     (bits & 15) == 0;
-#define FSIE_NORM_ROTATE(T, V)                                                                                      \
-    launch_dependent(norm_rotate_write_kernel<T, V>, dim3(tokens), dim3(warps * 32), smem, stream, (T*)proj, ld,    \
+#define FSIE_NORM_ROTATE(T)                                                                                        \
+    launch_dependent(norm_rotate_write_kernel<T>, dim3(tokens), dim3(warps * 32), smem, stream, (T*)proj, ld,       \
                      positions, cos_sin, table_len, slot_of, (T*)k_pages, (T*)v_pages, page_stride, page_size,     \
                      heads, kv_heads, dim, vdim, rotary_dim, q_gain, k_gain, eps, unit, whole, v_from_k, error)
-    if (dtype == DTYPE_F32) return vec ? FSIE_NORM_ROTATE(float, true) : FSIE_NORM_ROTATE(float, false);
-    return vec ? FSIE_NORM_ROTATE(bf16, true) : FSIE_NORM_ROTATE(bf16, false);
+    return dtype == DTYPE_F32 ? FSIE_NORM_ROTATE(float) : FSIE_NORM_ROTATE(bf16);
 #undef FSIE_NORM_ROTATE
 }
 

@@ -102,10 +102,10 @@ class DifferenceAttention(Mixer):
         tokens, wide = y.shape[0], MAPS * self.dim
         group = ctx.groups[cache.group]
         proj = rt.linear(y, self.w_in, None, "difference_attention.in")
-        # keys and values into their pages (nothing to rotate)
-        ops.rotate_mix_write(proj, ctx.positions, self.no_table, group.slot_of, cache.k_pages, cache.v_pages,
-                             cache.page_stride, group.page_size, self.heads, self.kv_heads, wide, self.vdim, 0, 0,
-                             None, None, ctx.error)
+        # keys and values into their pages (nothing to norm or rotate: the queries stay as they are)
+        ops.norm_rotate_write(proj, ctx.positions, self.no_table, group.slot_of, cache.k_pages, cache.v_pages,
+                              cache.page_stride, group.page_size, self.heads, self.kv_heads, wide, self.vdim, 0, None,
+                              None, self.eps, ctx.error)
         out = rt.buffer("difference_attention.out", tokens, self.heads * self.vdim, proj.dtype)
         gate0 = self.q_width + self.k_width + self.v_width
         gate = proj[:, gate0:gate0 + self.heads]

@@ -172,7 +172,9 @@ def run_attention(args, timer, decode: bool):
 
 
 def run_scaled_attention(args, timer):
-    """Attention with 32-bit weights, --softcap (0: none), chunks and a gate per column over shuffled pages."""
+    """Attention with 32-bit weights over shuffled pages: --softcap (0: none), chunks or a window, a gate per
+    column or per head, sinks; --maps 2: two keys side by side in a row, their ranges left for the merge of
+    differences, which is timed with it."""
     from ..parts.attention import attention_splits
     from ..parts.scaled_attention import key_splits
     heads, kv_heads, hd, page, new = args.heads, args.kv_heads, args.head_dim, args.page, args.tokens
@@ -181,7 +183,12 @@ def run_scaled_attention(args, timer):
     group, tokens = heads // kv_heads, batch * new
     wide = torch.randn(tokens, 2 * heads * hd, device="cuda").bfloat16()         # queries beside their gates
     gate = wide[:, heads * hd:] if args.gate else None
+    head_gate = wide[:, heads * hd:heads * hd + heads] if args.head_gate else None
+    maps, window = args.maps, args.window
+    if maps == 2:                                  # as many query heads for every map, half as wide
+        heads, group = 2 * heads, 2 * group
     scale = torch.full((heads,), hd ** -0.5, device="cuda")
+    sink = torch.randn(heads, device="cuda") if args.sink else None
     out = torch.empty(tokens, heads * hd, dtype=torch.bfloat16, device="cuda")
     error = torch.zeros(1, dtype=torch.int32, device="cuda")
     sms = torch.cuda.get_device_properties(0).multi_processor_count
@@ -190,27 +197,37 @@ def run_scaled_attention(args, timer):
     tiles.sort(key=lambda t: -t[1])
     i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")
     item, row0 = i32([t[0] for t in tiles]), i32([t[1] for t in tiles])
-    seen = lambda pos: pos % chunk + 1 if chunk else pos + 1
-    longest = min(args.context, chunk + per_tile) if chunk else args.context
+    seen = lambda pos: min(pos % chunk + 1 if chunk else pos + 1, window or pos + 1)
+    reach = chunk or window
+    longest = min(args.context, reach + per_tile) if reach else args.context
     nsplit = args.nsplit or (key_splits(len(tiles) * kv_heads, longest, sms, key_tile=64) if new == 1 else
                              attention_splits(len(tiles) * kv_heads, longest, sms, False, blocks_per_sm=1))
     parts = (torch.empty(nsplit * tokens * heads * hd, device="cuda"), torch.empty(nsplit * tokens * heads * 2, device="cuda"))
-    options = dict(chunk=chunk, softcap=args.softcap, gate=gate)
+    options = dict(chunk=chunk, softcap=args.softcap, gate=gate, sink=sink, maps=maps, partial=maps == 2,
+                   head_gate=None if maps == 2 else head_gate)
+
+    def merged(attention):
+        def run():
+            attention()
+            if maps == 2:
+                ops.difference_merge(*parts, out, tokens, heads // 2, hd, nsplit, 0.6, 1e-6, 0.4, head_gate)
+        return run
     if new == 1:
         slots = i32(list(range(batch)))
-        ms = timer(lambda: ops.scaled_attention(wide, wide.stride(0), scale, pages[:, 0, 0], pages[:, 0, 1], pages.stride(0),
-                                                page, hd, hd, False, tables, item, row0, len(tiles), qstart, qlen, pos0,
-                                                slots, out, tokens, heads, kv_heads, 0, error, nsplit, *parts,
-                                                form="mma_few", **options))
+        ms = timer(merged(lambda: ops.scaled_attention(
+            wide, wide.stride(0), scale, pages[:, 0, 0], pages[:, 0, 1], pages.stride(0), page, hd, hd, False, tables, item,
+            row0, len(tiles), qstart, qlen, pos0, slots, out, tokens, heads, kv_heads, window, error, nsplit, *parts,
+            form="mma_few", **options)))
     else:
         pages_map = ops.PagesMap(pages, "tc")
-        ms = timer(lambda: ops.attention_tc_scaled(pages_map, 0, wide, wide.stride(0), scale, tables, item, row0, len(tiles),
-                                                   qstart, qlen, pos0, out, tokens, heads, kv_heads, 0, error, nsplit,
-                                                   *parts, **options))
+        ms = timer(merged(lambda: ops.attention_tc_scaled(
+            pages_map, 0, wide, wide.stride(0), scale, tables, item, row0, len(tiles), qstart, qlen, pos0, out, tokens,
+            heads, kv_heads, window, error, nsplit, *parts, **options)))
     keys = sum(seen(past + t) for t in range(new))
     read = batch * min(args.context, seen(args.context - 1) if new == 1 else args.context)
     nbytes = 2 * (read * 2 * kv_heads * hd + tokens * heads * hd * (3 if args.gate else 2))
-    return ms, nbytes, 4.0 * heads * hd * batch * keys, {"nsplit": nsplit, "tiles": len(tiles), "error": int(error.item())}
+    # a query of two maps is half as wide as its key row
+    return ms, nbytes, (4.0 if maps == 1 else 3.0) * heads * hd * batch * keys, {"nsplit": nsplit, "tiles": len(tiles), "error": int(error.item())}
 
 
 def run_routed_experts(args, timer, dtype):
@@ -358,6 +375,66 @@ def run_state_space(args, timer, dtype):
                       "kernels": rows}))
 
 
+def run_gated_linear(args, timer, dtype):
+    """Every kernel of a gated linear attention mixer (--heads, --head-dim key columns, --vdim value columns, --rank)
+    over one prompt of --tokens, or over --batch requests with one token each, beside the same scan with one
+    decay per head at as many state numbers (heads of 128 x 128)."""
+    heads, dim, vdim, rank = args.heads, args.head_dim, args.vdim, args.rank
+    elem = 2 if dtype is torch.bfloat16 else 4
+    items = args.batch if args.tokens == 1 else 1
+    tokens = args.tokens * items
+    g = torch.Generator(device="cuda").manual_seed(0)
+    rand = lambda *shape: torch.randn(shape, generator=g, device="cuda", dtype=torch.float32)
+    dev = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")
+    qk, inner = heads * dim, heads * vdim
+    proj = (rand(tokens, -(-(2 * qk + 2 * inner + rank) // 8) * 8) * 0.5).to(dtype)
+    weight, bias, gain = rand(rank, qk) / rank ** 0.5, rand(qk), rand(vdim)
+    decay, o = torch.empty(tokens, qk, device="cuda"), torch.empty(tokens, inner, device="cuda")
+    y = torch.empty(tokens, inner, dtype=dtype, device="cuda")
+    per = args.tokens
+    qstart, qlen, slot = dev([i * per for i in range(items)]), dev([per] * items), dev(list(range(items)))
+    chunk = 64
+    segs = -(-per // chunk)
+
+    def chunks(floats):
+        if per <= 2 * chunk:
+            return {}
+        return dict(seg_item=dev([0] * segs), seg_row0=dev([i * chunk for i in range(segs)]), num_segs=segs,
+                    seg_tokens=chunk, chunk_states=torch.empty(segs * floats, device="cuda"))
+    peak, ffma, rows = peaks(), 148 * 128 * 2 * 1.965e9 / 1e12, []
+
+    def note(name, ms, nbytes, flops):
+        gbs, tflops = nbytes / (ms * 1e-3) / 1e9, flops / (ms * 1e-3) / 1e12
+        rows.append({"kernel": name, "ms": round(ms, 5), "GB/s": round(gbs, 1), "TFLOP/s": round(tflops, 2),
+                     "frac_hbm": round(gbs / peak["hbm_gbs"], 3), "frac_ffma": round(tflops / ffma, 3)})
+
+    note("row_decay", timer(lambda: ops.row_decay(proj, 2 * qk + 2 * inner, rank, weight, bias, 1 / 16.0, decay)),
+         tokens * (rank * elem + qk * 4), 2.0 * tokens * qk * rank)
+    matrix = heads * dim * vdim
+    state = torch.zeros(items, heads, dim, vdim, device="cuda")
+    options = chunks(matrix + qk)
+    carried = 2 * items * matrix * 4                         # the state in and out
+    note("lightning_scan, decay per state row", timer(lambda: ops.lightning_scan(
+        proj, 0, qk, 2 * qk, qstart, qlen, slot, items, state, None, o, heads, dim, vdim, decay_row=decay,
+        out_scale=dim ** -0.5, **options)),
+         tokens * ((2 * qk + inner) * elem + qk * 4 + inner * 4) * (2 if options else 1) + carried, 4.0 * tokens * matrix)
+    note("head_norm_silu", timer(lambda: ops.head_norm_silu(o, proj, 2 * qk + inner, gain, 1e-6, y, heads)),
+         tokens * inner * (4 + 2 * elem), 8.0 * tokens * inner)
+    like_heads = max(1, matrix // (128 * 128))
+    like, like_out = rand(tokens, 3 * like_heads * 128), torch.empty(tokens, like_heads * 128, device="cuda")
+    like_state = torch.zeros(items, like_heads, 128, 128, device="cuda")
+    like_decay = torch.linspace(0.9, 0.999, like_heads, device="cuda")
+    options = chunks(like_heads * 128 * 128)
+    note("lightning_scan, decay per head", timer(lambda: ops.lightning_scan(
+        like, 0, like_heads * 128, 2 * like_heads * 128, qstart, qlen, slot, items, like_state, like_decay, like_out,
+        like_heads, 128, 128, **options)),
+         tokens * 4 * like_heads * 128 * 4 * (2 if options else 1) + 2 * items * like_heads * 128 * 128 * 4,
+         4.0 * tokens * like_heads * 128 * 128)
+    print(json.dumps({"kernel": "gated_linear", "dtype": args.dtype, "tokens": tokens, "requests": items, "heads": heads,
+                      "dim": dim, "vdim": vdim, "rank": rank, "chunk_parallel": per > 2 * chunk, "peaks": peak["source"],
+                      "kernels": rows}))
+
+
 def run(args):
     timer = Timer(args.warmup, args.iters, not args.no_flush)
     dtype = torch.bfloat16 if args.dtype == "bfloat16" else torch.float32
@@ -454,6 +531,23 @@ def run(args):
         return run_routed_experts(args, timer, dtype)
     elif args.kernel == "state_space":
         return run_state_space(args, timer, dtype)
+    elif args.kernel == "gated_linear":
+        return run_gated_linear(args, timer, dtype)
+    elif args.kernel == "norm_rotate_write":
+        from ..parts.rope import rotary_table
+        heads, kv_heads, hd, page = args.heads, args.kv_heads, args.head_dim, args.page
+        own = 0 if args.keys_as_values else kv_heads * hd
+        qkv = rand(args.tokens, (heads + kv_heads) * hd + own + -(-heads // 8) * 8).to(dtype)
+        table = torch.from_numpy(rotary_table(1e6, hd // 2, args.tokens + 1)).cuda()
+        pages = torch.zeros((args.tokens // page + 1, 1, 2, kv_heads, page, hd), dtype=dtype, device="cuda")
+        pos = torch.arange(args.tokens, dtype=torch.int32, device="cuda")
+        error = torch.zeros(1, dtype=torch.int32, device="cuda")
+        q_gain, k_gain = (rand(heads * hd), rand(kv_heads * hd)) if args.whole_norm else (rand(hd), rand(hd))
+        ms = timer(lambda: ops.norm_rotate_write(qkv, pos, table, pos, pages[:, 0, 0], pages[:, 0, 1], pages.stride(0), page,
+                                                 heads, kv_heads, hd, hd, hd // 2, q_gain, k_gain, 1e-6, error,
+                                                 whole=args.whole_norm, values_from_keys=args.keys_as_values))
+        nbytes = args.tokens * elem * (2 * heads * hd + 3 * kv_heads * hd + own)
+        flops = 10.0 * args.tokens * (heads + kv_heads) * hd
     elif args.kernel == "scaled_attention":
         ms, nbytes, flops, extra = run_scaled_attention(args, timer)
     elif args.kernel == "stream_norm":
@@ -462,7 +556,9 @@ def run(args):
         mix, spread, gather = torch.eye(s, device="cuda") + 0.01 * rand(s, s), rand(s) * 0.1, rand(s)
         gain, bias = rand(args.hidden), rand(args.hidden)
         out = torch.empty((args.tokens, args.hidden), dtype=dtype, device="cuda")
-        ms = timer(lambda: ops.stream_norm(x, None, y, mix, spread, gather, gain, bias, 1e-6, out))
+        scale = rand(args.hidden) if args.scaled else None
+        ms = timer(lambda: ops.stream_norm(x, None, y, mix, spread, gather, gain, None if args.scaled else bias, 1e-6, out,
+                                           centred=not args.scaled, delta_scale=scale))
         nbytes, flops = args.tokens * args.hidden * (8 * s + 2 * elem), 2.0 * args.tokens * args.hidden * s * (s + 2)
     elif args.kernel == "sum_layernorm":
         x, d1, d2 = rand(args.tokens, args.hidden), rand(args.tokens, args.hidden).to(dtype), \
@@ -508,6 +604,16 @@ def main(argv=None) -> int:
     parser.add_argument("--chunk", type=int, default=0, help="scaled_attention: positions per chunk (0: none)")
     parser.add_argument("--softcap", type=float, default=0.0, help="scaled_attention: cap on the scores (0: none)")
     parser.add_argument("--gate", action="store_true", help="scaled_attention: a gate per column")
+    parser.add_argument("--head-gate", action="store_true", help="scaled_attention: a gate per head")
+    parser.add_argument("--sink", action="store_true", help="scaled_attention: a sink per head")
+    parser.add_argument("--window", type=int, default=0, help="scaled_attention: keys a query sees (0: all)")
+    parser.add_argument("--maps", type=int, default=1, choices=[1, 2],
+                        help="scaled_attention: 2 = two keys of half the head size, with the merge of differences")
+    parser.add_argument("--vdim", type=int, default=128, help="gated_linear: value columns per head")
+    parser.add_argument("--rank", type=int, default=16, help="gated_linear: width of the narrow product of the decays")
+    parser.add_argument("--whole-norm", action="store_true", help="norm_rotate_write: the norm over all heads at once")
+    parser.add_argument("--keys-as-values", action="store_true", help="norm_rotate_write: values are the keys as projected")
+    parser.add_argument("--scaled", action="store_true", help="stream_norm: outputs scaled by column, RMS norm")
     parser.add_argument("--experts", type=int, default=64)
     parser.add_argument("--top", type=int, default=6)
     parser.add_argument("--groups", type=int, default=8)

@@ -54,9 +54,10 @@ LIBRARIES: Dict[str, Sequence[str]] = {
     # cache of latent rows
     "mixers": ("sandwich_norm.cu", "mingru.cu", "scaled_attention.cu", "latent_attention.cu"),
     # decoders whose sublayers share one norm: layer norm with gain and bias over a sum of pending
-    # outputs, the residual stream beside the embedding output, capped logits, a sigmoid gate; and a
-    # feed-forward of routed experts
-    "routed": ("parallel_norm.cu", "routed.cu"),
+    # outputs, the residual stream beside the embedding output, scaled and capped logits, a sigmoid gate
+    "parallel": ("parallel_norm.cu",),
+    # a feed-forward of routed experts
+    "routed": ("routed.cu",),
     # residuals of several streams that every sublayer reads and writes through small matrices
     "streams": ("stream_norm.cu",),
 }

@@ -42,6 +42,14 @@ class PinnedRing:
         self.next = 0
         self.bytes_staged = 0        # host-to-device bytes so far (benchmarks read this)
 
+    def _grow(self, ints: int) -> None:
+        """All buffers anew with room for `ints` each, in one pinned piece: pinning is slow, and one by
+        one it would fall into the first `depth` stagings of a serving run."""
+        for event in self.events:
+            if event is not None:
+                event.synchronize()
+        self.buffers = list(torch.empty(self.depth * ints, dtype=torch.int32, pin_memory=True).split(ints))
+
     def stage(self, host: np.ndarray, device: torch.device,
               out: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Copy `host` (int32) to the device; into the front of `out` when given (a fixed
@@ -52,7 +60,7 @@ class PinnedRing:
             self.events[i].synchronize()
         n = host.size
         if self.buffers[i] is None or self.buffers[i].numel() < n:
-            self.buffers[i] = torch.empty(max(n, 1024) * 2, dtype=torch.int32).pin_memory()
+            self._grow(max(n, 1024) * 2)
         staging = self.buffers[i][:n]
         staging.numpy()[:] = host
         self.bytes_staged += n * 4

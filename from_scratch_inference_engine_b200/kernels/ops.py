@@ -1750,30 +1750,42 @@ def head_product(x: torch.Tensor, x_ld: int, x_head: int, weight: torch.Tensor, 
 
 
 # ------------------------------------------------- one norm for two sublayers; routed experts
+_parallel = None
 _routed = None
 
 
-def routed():
-    """The library of decoders whose sublayers share one norm and whose feed-forward is a set of
-    routed experts (layer norm with gain and bias over a sum of pending outputs, the residual stream
-    beside the embedding output, a cap on the logits, a sigmoid gate; router, sorting of the
-    (token, expert) pairs, the experts' products, the weighted sum), compiled at first use."""
-    global _routed
-    if _routed is None:
-        lib = build.load_library("routed")
+def parallel():
+    """The library of decoders whose sublayers share one norm (layer norm with gain and bias over a sum
+    of pending outputs, the residual stream beside the embedding output, a scale and a cap on the
+    logits, a sigmoid gate), compiled at first use."""
+    global _parallel
+    if _parallel is None:
+        lib = build.load_library("parallel")
         i, f, ll, p = ctypes.c_int, ctypes.c_float, ctypes.c_longlong, ctypes.c_void_p
         lib.fsie_sum_layernorm.argtypes = [p, p, p, p, p, p, p, i, i, f, i, i, p]
         lib.fsie_settle_concat.argtypes = [p, p, p, p, p, i, i, i, p]
         lib.fsie_logit_cap.argtypes = [p, ll, f, f, p]
         lib.fsie_sigmoid_gate.argtypes = [p, i, p, i, i, i, i, p]
+        for name in ("fsie_sum_layernorm", "fsie_settle_concat", "fsie_logit_cap", "fsie_sigmoid_gate"):
+            getattr(lib, name).restype = i
+        _parallel = lib
+    return _parallel
+
+
+def routed():
+    """The library of feed-forwards of routed experts (router, sorting of the (token, expert) pairs, the
+    experts' products, the weighted sum), compiled at first use."""
+    global _routed
+    if _routed is None:
+        lib = build.load_library("routed")
+        i, f, ll, p = ctypes.c_int, ctypes.c_float, ctypes.c_longlong, ctypes.c_void_p
         lib.fsie_moe_tile_rows.argtypes = []
         lib.fsie_moe_route.argtypes = [p, i, p, p, p, p, p, p, i, i, i, i, i, i, f, i, i, i, i, p]
         lib.fsie_moe_align.argtypes = [p, i, i, i, i, p, p, p, p, p, p, p]
         lib.fsie_moe_gather.argtypes = [p, ll, p, p, i, i, p, i, i, p]
         lib.fsie_moe_product.argtypes = [p, ll, p, p, ll, p, p, p, p, p, i, i, i, i, i, i, i, i, p]
         lib.fsie_moe_combine.argtypes = [p, p, p, p, p, i, i, i, p, i, p, ll, i, p]
-        for name in ("fsie_sum_layernorm", "fsie_settle_concat", "fsie_logit_cap", "fsie_sigmoid_gate",
-                     "fsie_moe_tile_rows", "fsie_moe_route", "fsie_moe_align", "fsie_moe_gather", "fsie_moe_product",
+        for name in ("fsie_moe_tile_rows", "fsie_moe_route", "fsie_moe_align", "fsie_moe_gather", "fsie_moe_product",
                      "fsie_moe_combine"):
             getattr(lib, name).restype = i
         _routed = lib
@@ -1815,7 +1827,7 @@ def sum_layernorm(x: torch.Tensor, deltas, gain: Optional[torch.Tensor], bias: O
         raise KernelError("sum_layernorm: out is too small")
     d1 = deltas[0] if deltas else None
     d2 = deltas[1] if len(deltas) > 1 else None
-    _check(routed().fsie_sum_layernorm(_ptr(x), _ptr(d1), _ptr(d2), _ptr(gain), _ptr(bias), _ptr(rows),
+    _check(parallel().fsie_sum_layernorm(_ptr(x), _ptr(d1), _ptr(d2), _ptr(gain), _ptr(bias), _ptr(rows),
                                        _ptr(out), count, width, float(eps), int(write_x), _tag(dtype),
                                        _stream()), "sum_layernorm")
     return out
@@ -1837,7 +1849,7 @@ def settle_concat(x: torch.Tensor, deltas, x0: torch.Tensor, out: torch.Tensor) 
             raise KernelError("settle_concat: a pending output is not of x's shape")
     d1 = deltas[0] if deltas else None
     d2 = deltas[1] if len(deltas) > 1 else None
-    _check(routed().fsie_settle_concat(_ptr(x), _ptr(d1), _ptr(d2), _ptr(x0), _ptr(out), tokens, width,
+    _check(parallel().fsie_settle_concat(_ptr(x), _ptr(d1), _ptr(d2), _ptr(x0), _ptr(out), tokens, width,
                                        _tag(out.dtype), _stream()), "settle_concat")
     return out
 
@@ -1845,7 +1857,7 @@ def settle_concat(x: torch.Tensor, deltas, x0: torch.Tensor, out: torch.Tensor) 
 def logit_cap(logits: torch.Tensor, scale: float, cap: float) -> torch.Tensor:
     """logits <- cap * tanh(logits * scale / cap) in place (cap = 0: logits * scale)."""
     _need(logits, torch.float32, "logits")
-    _check(routed().fsie_logit_cap(_ptr(logits), logits.numel(), float(scale), float(cap), _stream()),
+    _check(parallel().fsie_logit_cap(_ptr(logits), logits.numel(), float(scale), float(cap), _stream()),
            "logit_cap")
     return logits
 
@@ -1858,7 +1870,7 @@ def sigmoid_gate(out: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
     tokens, width = out.shape
     if gate.shape != out.shape or out.stride(1) != 1 or gate.stride(1) != 1:
         raise KernelError("sigmoid_gate: shapes do not fit")
-    _check(routed().fsie_sigmoid_gate(_ptr(out), out.stride(0), _ptr(gate), gate.stride(0), tokens, width,
+    _check(parallel().fsie_sigmoid_gate(_ptr(out), out.stride(0), _ptr(gate), gate.stride(0), tokens, width,
                                       _tag(out.dtype), _stream()), "sigmoid_gate")
     return out
 

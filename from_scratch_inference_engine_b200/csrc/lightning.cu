@@ -43,7 +43,7 @@ __device__ __forceinline__ void scan_store4(bf16* p, float4 v) {
 // where row d of a staged q or k vector lives: the DR rows of a thread are contiguous (one or
 // more 16-byte loads) and the groups are four floats apart in the banks
 template <int DR> __device__ __forceinline__ int scan_row_at(int d) {
-    constexpr int PAD = DR >= 4 ? DR + 4 : DR;
+    constexpr int PAD = DR > 4 ? DR + 4 : DR;
     return (d / DR) * PAD + d % DR;
 }
 
@@ -71,7 +71,7 @@ lightning_scan_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off, 
                       float out_scale, long long state_stride, float* __restrict__ chunk_decay) {
     // tokens staged in shared memory at a time (fewer where q, k and the rows' decays of large heads are staged)
     constexpr int SCAN_TOKENS = ROWS && DR > 8 ? 8 : 16;
-    constexpr int PAD = DR >= 4 ? DR + 4 : DR;
+    constexpr int PAD = DR > 4 ? DR + 4 : DR;
     constexpr int ROW_LEN = SCAN_ROW_GROUPS * PAD;
     __shared__ __align__(16) float qs[SCAN_TOKENS * ROW_LEN];
     __shared__ __align__(16) float ks[SCAN_TOKENS * ROW_LEN];

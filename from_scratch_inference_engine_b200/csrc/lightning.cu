@@ -283,13 +283,19 @@ __global__ void lightning_chain_kernel(const int* __restrict__ item_qstart, cons
 
 // The decays of gated linear attention: a = sigmoid(z)^(1/tau) with z = low W^T + bias, low the token's `rank`
 // columns of proj at low_off, W given as wt [rank, columns].  Through the logarithm, log sigmoid(z) = min(z, 0)
-// - log(1 + e^-|z|), in 32-bit.  A thread owns a column of DECAY_TOKENS tokens: a weight is fetched once for all.
-constexpr int DECAY_TOKENS = 16;
+// - log(1 + e^-|z|), in 32-bit: what rounding 1 + e^-|z| loses is below a rounding of the result.  A thread owns a column of DECAY_TOKENS tokens: a weight is fetched once for all.
+// The first DECAY_AHEAD of them are asked for while the kernel before still runs.
+constexpr int DECAY_TOKENS = 16, DECAY_AHEAD = 16;
 template <typename T>
-__global__ void row_decay_kernel(const T* __restrict__ proj, int ld, int low_off, int rank, const float* __restrict__ wt,
-                                 const float* __restrict__ bias, float inv_tau, float* __restrict__ out, int tokens,
-                                 int columns) {
+__global__ void __launch_bounds__(128) row_decay_kernel(
+        const T* __restrict__ proj, int ld, int low_off, int rank, const float* __restrict__ wt,
+        const float* __restrict__ bias, float inv_tau, float* __restrict__ out, int tokens, int columns) {
     extern __shared__ __align__(16) float rd_low[];      // [rank][DECAY_TOKENS]
+    const int c = blockIdx.x * blockDim.x + threadIdx.x;
+    float w[DECAY_AHEAD];
+#pragma unroll
+    for (int r = 0; r < DECAY_AHEAD; ++r) w[r] = r < rank && c < columns ? wt[(size_t)r * columns + c] : 0.f;
+    const float b = c < columns ? bias[c] : 0.f;
     grid_dependency_wait();
     grid_dependents_go();
     const int t0 = blockIdx.y * DECAY_TOKENS;
@@ -299,30 +305,36 @@ __global__ void row_decay_kernel(const T* __restrict__ proj, int ld, int low_off
         rd_low[r * DECAY_TOKENS + t] = t < n ? to_float(proj[(size_t)(t0 + t) * ld + low_off + r]) : 0.f;
     }
     __syncthreads();
-    const int c = blockIdx.x * blockDim.x + threadIdx.x;
     if (c >= columns) return;
     float z[DECAY_TOKENS];
-    const float b = bias[c];
 #pragma unroll
     for (int t = 0; t < DECAY_TOKENS; ++t) z[t] = b;
-#pragma unroll 4
-    for (int r = 0; r < rank; ++r) {
-        const float w = wt[(size_t)r * columns + c];
-        const float4* low = reinterpret_cast<const float4*>(rd_low + r * DECAY_TOKENS);
+    for (int r0 = 0; r0 < rank; r0 += DECAY_AHEAD) {
 #pragma unroll
-        for (int q = 0; q < DECAY_TOKENS / 4; ++q) {
-            const float4 v = low[q];
-            z[4 * q] = fmaf(w, v.x, z[4 * q]);
-            z[4 * q + 1] = fmaf(w, v.y, z[4 * q + 1]);
-            z[4 * q + 2] = fmaf(w, v.z, z[4 * q + 2]);
-            z[4 * q + 3] = fmaf(w, v.w, z[4 * q + 3]);
+        for (int j = 0; j < DECAY_AHEAD; ++j) {
+            if (r0 + j >= rank) break;
+            const float4* low = reinterpret_cast<const float4*>(rd_low + (r0 + j) * DECAY_TOKENS);
+#pragma unroll
+            for (int q = 0; q < DECAY_TOKENS / 4; ++q) {
+                const float4 v = low[q];
+                z[4 * q] = fmaf(w[j], v.x, z[4 * q]);
+                z[4 * q + 1] = fmaf(w[j], v.y, z[4 * q + 1]);
+                z[4 * q + 2] = fmaf(w[j], v.z, z[4 * q + 2]);
+                z[4 * q + 3] = fmaf(w[j], v.w, z[4 * q + 3]);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < DECAY_AHEAD; ++j) {
+            const int r = r0 + DECAY_AHEAD + j;
+            if (r < rank) w[j] = wt[(size_t)r * columns + c];
         }
     }
+    float* dst = out + (size_t)t0 * columns + c;
 #pragma unroll
-    for (int t = 0; t < DECAY_TOKENS; ++t) {
-        if (t >= n) break;
-        const float log_sigmoid = fminf(z[t], 0.f) - log1pf(expf(-fabsf(z[t])));
-        out[(size_t)(t0 + t) * columns + c] = expf(log_sigmoid * inv_tau);
+    for (int t = 0; t < DECAY_TOKENS; ++t, dst += columns) {
+        const float log_sigmoid = fminf(z[t], 0.f) - logf(1.0f + __expf(-fabsf(z[t])));
+        const float a = expf(log_sigmoid * inv_tau);
+        if (t < n) *dst = a;
     }
 }
 

@@ -576,13 +576,13 @@ def lanilorn_shapes(width, heads, kv_heads, dim, streams, ff, gla_heads, gla_dim
     kinds = ("attention_2", "attention", "gla", "attention")
     heads_of = {"heads": heads, "kv_heads": kv_heads, "vdim": dim, "scale": dim ** -0.5}
     mixers = {"attention": dict(heads_of, dim=dim, mask={"size": window}, rot={
-                  "base": 250000.0, "dims": dim // 2,
-                  "scaling": {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}}),
-              "attention_2": dict(heads_of, dim=dim // 2, diff=0.6, q_temp={"coef": 0.3, "every": 64}),
+                  "base": 500000.0, "dims": dim // 2,
+                  "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}),
+              "attention_2": dict(heads_of, dim=dim // 2, diff=0.5, q_temp={"coef": 0.1, "every": 4096}),
               "gla": {"heads": gla_heads, "dim": gla_dim, "vdim": gla_vdim, "tau": 16.0}}
     order = [kinds[i % len(kinds)] for i in range(layers)]
     lanilorn = {"architecture": "Lanilorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
-                "streams": streams, "embedding": {"scale": 0.5}, "logit_scale": 0.25,
+                "streams": streams, "embedding": {"scale": 2.0}, "logit_scale": 0.5,
                 "layers": [{"type": kind, "mixer": mixers[kind],
                             "mlp": None if kind == "gla" else {"kind": "dense", "ff": ff}} for kind in order]}
     beside = {"attention": dict(heads_of, dim=dim, mask={"size": 2 * window}), "full": dict(heads_of, dim=dim)}

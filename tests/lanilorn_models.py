@@ -74,10 +74,10 @@ CONFIGS = {
     "wide": model(150, 128, 1e-3, 3, [
         layer(difference(4, 2, 32, 64, 1.2, 0.4, 0.2, 32), 192),
         layer(attention(4, 1, 64, 100, 0.35, yarn(20000.0, 32, 4.0, 128, 32.0, 1.0)), 256),
-        layer(gla(2, 64, 64, 16.0, 16)),
-        layer(difference(2, 1, 64, 128, 0.8, 0.6, 0.3, 64), 128),
+        layer(gla(2, 64, 64, 12.0, 24)),
+        layer(difference(2, 1, 64, 128, 0.8, 0.7, 0.25, 80), 128),
         layer(attention(4, 2, 128, 56, 0.25, yarn(20000.0, 128, 2.0, 64, 32.0, 1.0)), 64),
-        layer(difference(4, 4, 48, 96, 0.9, 0.5, 0.3, 20))]),
+        layer(difference(6, 3, 48, 96, 0.9, 0.5, 0.35, 20))]),
 }
 
 

@@ -293,7 +293,7 @@ LENGTHS = [(300, 177), (0, 90), (40, 2), (260, 1)]
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("dim,heads,kv_heads,window,page", [
-    (24, 6, 2, 37, 16), (96, 4, 1, 50, 8), (32, 6, 6, 1, 16), (64, 8, 2, 100, 32), (128, 6, 3, 129, 16), (128, 8, 1, 0, 16)])
+    (24, 6, 2, 37, 16), (96, 4, 1, 50, 8), (32, 6, 6, 1, 16), (64, 8, 2, 100, 32), (128, 6, 3, 129, 16), (128, 10, 1, 0, 16)])
 def test_windows_sinks_and_gates_per_head(dtype, dim, heads, kv_heads, window, page):
     """Every form of the attention kernel that takes the sizes, whole and split over key ranges: a long
     portion behind 300 cached tokens, a first portion, two tokens behind 40, a token decoded at position
@@ -309,7 +309,7 @@ def test_windows_sinks_and_gates_per_head(dtype, dim, heads, kv_heads, window, p
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("dim,dv,heads,kv_heads,page", [
-    (12, 20, 4, 2, 16), (7, 5, 3, 1, 16), (48, 96, 4, 4, 8), (16, 32, 6, 3, 16), (32, 64, 8, 2, 16), (64, 128, 4, 1, 32),
+    (12, 20, 4, 2, 16), (7, 5, 3, 1, 16), (48, 96, 6, 2, 8), (16, 32, 6, 3, 16), (32, 64, 8, 2, 16), (64, 128, 4, 1, 32),
     (64, 128, 4, 4, 16), (48, 192, 2, 2, 16), (8, 400, 2, 1, 16)])
 def test_the_difference_of_two_maps(dtype, dim, dv, heads, kv_heads, page):
     """Every form of the attention over two keys side by side, its ranges merged, subtracted, normed and gated:
@@ -364,7 +364,7 @@ def test_decays_through_their_logarithms(dtype, rank, columns, tokens):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("heads,dim,vdim", [(3, 10, 14), (2, 32, 32), (1, 64, 128), (2, 100, 36), (2, 200, 20), (1, 256, 64)])
+@pytest.mark.parametrize("heads,dim,vdim", [(3, 10, 14), (3, 32, 40), (1, 64, 128), (2, 100, 36), (2, 200, 20), (1, 256, 64)])
 def test_scan_with_a_decay_per_state_row(dtype, heads, dim, vdim):
     """Two requests' tokens as one batch - in one call, in three that carry the state, and chunk by
     chunk - against the recurrence token by token; slots in another order than the requests, one slot

@@ -160,11 +160,11 @@ def test_tables_of_angles_and_temperatures():
         for i, f in enumerate(freq):
             assert abs(table[p, i] - magnitude * math.cos(p * f)) < 1e-6
             assert abs(table[p, 6 + i] - magnitude * math.sin(p * f)) < 1e-6
-    for coef, every in ((0.3, 64), (0.5, 1), (0.2, 7)):
+    for coef, every in ((0.25, 48), (0.5, 1), (0.2, 7)):
         want = plain.query_temperature(200, {"coef": coef, "every": every}).numpy()
         assert np.abs(query_temperature_table(coef, every, 200) - want).max() < 1e-6
     # the first step of the temperature falls on position every - 1
-    assert query_temperature_table(0.3, 64, 70)[62] == 1.0 and query_temperature_table(0.3, 64, 70)[63] > 1.2
+    assert query_temperature_table(0.25, 48, 70)[46] == 1.0 and query_temperature_table(0.25, 48, 70)[47] > 1.17
 
 
 def test_plain_mechanisms():
